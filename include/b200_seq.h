@@ -122,12 +122,13 @@ int b200_seq_cast_rows(const float* x, void* out, int dt, int64_t n, void* strea
 /* rows [g | u] (type dt, 2F wide) -> act(g) * u; act 0: SiLU, 1: GELU in its tanh form */
 int b200_seq_ff_gate(const void* gu, void* out, int dt, int64_t rows, int64_t F, int act, void* stream);
 /* gated delta rule over fp32 state slots S [slots, H, dk, dv]: per token S <- g S, u = beta (v - S^T k), S <- S + k u^T, y = S^T q; q and k
- * (kv_heads x dk, shared by H / kv_heads heads) are made unit vectors, q times q_scale; beta = sigmoid(raw[col_b + h]),
- * g = exp(-exp(A_log[h]) softplus(raw[col_a + h] + dt_bias[h])); c holds the activated q / k / v columns; y fp32 [T, H * dv] */
-int b200_seq_delta_scan(const float* c, int64_t ldc, int col_q, int col_k, int col_v, const float* raw, int64_t ldr, int col_b, int col_a,
-                        const void* A_log, const void* dt_bias, int dt, float q_scale, float* S_state, const int32_t* state_slots,
-                        const int32_t* cu_q, const int64_t* position_ids, float* y, int64_t ld_y, int B, int H, int kv_heads, int dk, int dv,
-                        void* stream);
+ * (kv_heads x dk, shared by H / kv_heads heads) are made unit vectors, q times q_scale; beta = sigmoid(raw[col_b + h]); decay per head,
+ * g = exp(-exp(A_log[h]) softplus(dec[col_a + h] + dt_bias[h])), or (channels != 0) per head and key channel n, acting on row n of S,
+ * g = exp(-exp(A_log[h]) softplus(dec[col_a + h dk + n] + dt_bias[h dk + n])); c holds the activated q / k / v columns; y fp32 [T, H * dv] */
+int b200_seq_delta_scan(const float* c, int64_t ldc, int col_q, int col_k, int col_v, const float* raw, int64_t ldr, int col_b, const float* dec,
+                        int64_t ldd, int col_a, int channels, const void* A_log, const void* dt_bias, int dt, float q_scale, float* S_state,
+                        const int32_t* state_slots, const int32_t* cu_q, const int64_t* position_ids, float* y, int64_t ld_y, int B, int H,
+                        int kv_heads, int dk, int dv, void* stream);
 /* per token: RMS norm over the whole q projection (H * d columns) and the whole k projection (G * d) when whole_norm != 0 (weights per
  * column, may be NULL), rotation of the first `rot` columns of every head, column i paired with i + rot / 2 (cos / sin fp32
  * [positions, rot / 2]); keys and values to the token-major cache row [k_off: G * d | v_off: G * dv], queries to q_out fp32 [T, H * d].
@@ -153,8 +154,14 @@ int b200_seq_talk_attn_splits(int dt, int64_t T, int B, int H, int G, int d, int
  * u / sqrt(mean u^2 + eps) * w (w of type dt; NULL: typed <- u) */
 int b200_seq_streams_step(float* X, int S, const float* init, const float* y, const float* mix, const float* out_coef, const float* in_coef,
                           const void* w, int dt, void* typed, int64_t T, int64_t W, float eps, void* stream);
+/* one fp32 stream between two sublayers, x [T, W] in place (or from `init`, then x is only written): x += y_scale * (n(y1) + n(y2)) with
+ * n(y) = y / sqrt(mean y^2 + eps) * w (w of type dt; NULL: n(y) = y; y1, y2 fp32 [T, W], may be NULL), then x += add (fp32 [T, W], may be
+ * NULL) + step_vec (type dt, [W], may be NULL), then typed (type dt) <- x / sqrt(mean x^2 + eps) * norm_w (norm_w NULL: not written) */
+int b200_seq_branches_step(float* x, const float* init, const float* y1, const void* w1, const float* y2, const void* w2, float y_scale,
+                           const float* add, const void* step_vec, const void* norm_w, int dt, void* typed, int64_t T, int64_t W, float eps,
+                           void* stream);
 /* out (dense rows of type out_dt) = act(in) over rows of F columns with leading dimension ld_in; act 0: SiLU, 1: GELU in its tanh form,
- * 2: tanh; element types fp32 -> any or bf16 -> bf16 */
+ * 2: tanh, 3: relu(z)^2, 4: none (a copy or a change of type); element types fp32 -> any or bf16 -> bf16 */
 int b200_seq_ff_act(const void* in, int in_dt, int64_t ld_in, void* out, int out_dt, int64_t rows, int64_t F, int act, void* stream);
 /* a fp32 [T, H, dv]: the first `rot` columns of every head turn by minus the token's position (cos / sin fp32 [positions, rot / 2]; pairs
  * as in b200_seq_qk_rot_prepare's values), the head is multiplied by sigmoid(gate[t * ld_gate + h]) (gate NULL: by 1) and by out_scale

@@ -1,8 +1,8 @@
 // Row kernels around an fp32 residual stream: embedding lookup (scaled, or plus a learned position row), layer norm in and out of
 // the stream, RMS norm of the stream with an offset weight, RMS norm of a
 // column slice, grouped RMS norm with a gate, the clamped gated feed-forward activation, the per-layer token side input, the step
-// between two sublayers of a decoder with several residual streams (write all streams, read and norm the next input), plain
-// activations, and the turn-back + gate of attention heads whose values carry their position.
+// between two sublayers of a decoder with several residual streams (write all streams, read and norm the next input) and of one
+// whose sublayers have one or two branches, each with a norm of its own, plain activations, and the turn-back + gate of attention heads whose values carry their position.
 // One block per token row; all statistics and the residual sum in fp32.
 #include "seq_common.cuh"
 
@@ -322,8 +322,107 @@ __global__ void __launch_bounds__(kRowThreads) streams_step_kernel(float* __rest
   }
 }
 
+// One stream between two sublayers (row t of x, fp32):
+//   r = (init ? init[t] : x[t]) + y_scale * (n_1(y1[t]) + n_2(y2[t])) + add[t] + step_vec,   n_i(y) = y / sqrt(mean(y^2) + eps) * w_i
+// (w_i NULL: the branch is added as it is; any term may be missing), x[t] <- r, typed[t] <- r / sqrt(mean(r^2) + eps) * norm_w.
+// One block per token; the branches' rows and r wait in shared memory between the passes (every thread reads back what it wrote).
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kRowThreads) branches_step_kernel(float* __restrict__ x, const float* __restrict__ init, const float* __restrict__ y1,
+                                                                    const T* __restrict__ w1, const float* __restrict__ y2, const T* __restrict__ w2,
+                                                                    float y_scale, const float* __restrict__ add, const T* __restrict__ step_vec,
+                                                                    const T* __restrict__ norm_w, T* __restrict__ typed, int W, float eps) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) float rows[];
+  __shared__ float red[3][32];
+  const int64_t t = blockIdx.x;
+  const int pitch = (W + 3) & ~3;
+  float *row = rows, *r1 = rows + pitch, *r2 = r1 + pitch;
+  float q1 = 0.f, q2 = 0.f;
+  for (int i = threadIdx.x * VEC; i < W; i += kRowThreads * VEC) {
+    float r[VEC], v[VEC];
+    ld_vec<VEC>((init ? init : x) + t * W + i, r);
+    if (add) {
+      ld_vec<VEC>(add + t * W + i, v);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) r[k] += v[k];
+    }
+    if (step_vec) {
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) r[k] += ldf(step_vec + i + k);
+    }
+    st_vec<float, VEC>(row + i, r);
+    if (y1) {
+      ld_vec<VEC>(y1 + t * W + i, v);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) q1 += v[k] * v[k];
+      st_vec<float, VEC>(r1 + i, v);
+    }
+    if (y2) {
+      ld_vec<VEC>(y2 + t * W + i, v);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) q2 += v[k] * v[k];
+      st_vec<float, VEC>(r2 + i, v);
+    }
+  }
+  float s1 = y_scale, s2 = y_scale;
+  if (w1 || w2) {   // both statistics behind one barrier
+    q1 = warp_sum(q1);
+    q2 = warp_sum(q2);
+    if (lane_id() == 0) {
+      red[0][warp_id()] = q1;
+      red[1][warp_id()] = q2;
+    }
+    __syncthreads();
+    constexpr int kWarps = kRowThreads / 32;
+    q1 = warp_sum(lane_id() < kWarps ? red[0][lane_id()] : 0.f);
+    q2 = warp_sum(lane_id() < kWarps ? red[1][lane_id()] : 0.f);
+    if (w1) s1 *= 1.f / sqrtf(q1 / W + eps);
+    if (w2) s2 *= 1.f / sqrtf(q2 / W + eps);
+  }
+  float q = 0.f;
+  for (int i = threadIdx.x * VEC; i < W; i += kRowThreads * VEC) {
+    float r[VEC], v[VEC];
+    ld_vec<VEC>(row + i, r);
+    if (y1) {
+      ld_vec<VEC>(r1 + i, v);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) r[k] = fmaf(s1 * v[k], w1 ? ldf(w1 + i + k) : 1.f, r[k]);
+    }
+    if (y2) {
+      ld_vec<VEC>(r2 + i, v);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) r[k] = fmaf(s2 * v[k], w2 ? ldf(w2 + i + k) : 1.f, r[k]);
+    }
+    st_vec<float, VEC>(x + t * W + i, r);
+    if (norm_w) {
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) q += r[k] * r[k];
+      st_vec<float, VEC>(row + i, r);
+    }
+  }
+  if (!norm_w) return;
+  const float rstd = 1.f / sqrtf(block_sum(q, red[2]) / W + eps);
+  for (int i = threadIdx.x * VEC; i < W; i += kRowThreads * VEC) {
+    float r[VEC];
+    ld_vec<VEC>(row + i, r);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) r[k] *= rstd * ldf(norm_w + i + k);
+    st_vec<T, VEC>(typed + t * W + i, r);
+  }
+}
+
 // out = act(in) element by element over rows of F columns (in may be a column slice: leading dimension ld_in);
-// act 0: SiLU, 1: GELU (tanh form), 2: tanh.  Evaluated in fp32.
+// act 0: SiLU, 1: GELU (tanh form), 2: tanh, 3: relu squared, 4: none (a copy or a change of type).  Evaluated in fp32.
+template <int ACT>
+__device__ __forceinline__ float plain_act_f(float z) {
+  if constexpr (ACT == 0) return silu_f(z);
+  else if constexpr (ACT == 1) return gelu_tanh_f(z);
+  else if constexpr (ACT == 2) return tanhf(z);
+  else if constexpr (ACT == 3) { const float p = fmaxf(z, 0.f); return p * p; }
+  else return z;
+}
+
 template <typename TI, typename TO, int ACT>
 __global__ void ff_act_kernel(const TI* __restrict__ in, int64_t ld_in, TO* __restrict__ out, int64_t rows, int F) {
   pdl_launch_dependents();
@@ -332,7 +431,7 @@ __global__ void ff_act_kernel(const TI* __restrict__ in, int64_t ld_in, TO* __re
   for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
     const int64_t r = i / F, c = i % F;
     const float z = ldf(in + r * ld_in + c);
-    stf(out + i, ACT == 1 ? gelu_tanh_f(z) : (ACT == 2 ? tanhf(z) : silu_f(z)));
+    stf(out + i, plain_act_f<ACT>(z));
   }
 }
 
@@ -543,18 +642,48 @@ extern "C" int b200_seq_streams_step(float* X, int S, const float* init, const f
   return B200_OK;
 }
 
-// in: rows of type in_dt (leading dimension ld_in), out: dense rows of type out_dt; act 0 SiLU, 1 GELU (tanh form), 2 tanh
+// x fp32 [T, W] in place, or from `init` [T, W]; y1 / y2 fp32 [T, W] with optional norm weights w1 / w2 [W]; add fp32 [T, W], step_vec [W]; norm_w
+// [W] with typed [T, W]; every pointer but x may be NULL.  Weights, step_vec and typed of element type dt.
+extern "C" int b200_seq_branches_step(float* x, const float* init, const float* y1, const void* w1, const float* y2, const void* w2, float y_scale,
+                                      const float* add, const void* step_vec, const void* norm_w, int dt, void* typed, int64_t T, int64_t W,
+                                      float eps, void* stream) {
+  if (T == 0) return B200_OK;
+  if (W > 13000 || (norm_w && !typed) || (w1 && !y1) || (w2 && !y2)) {
+    b200_set_last_error("seq_branches_step: width <= 13000; a norm needs its row");
+    return B200_ERR_ARG;
+  }
+  const size_t smem = (size_t)((W + 3) & ~3) * 4 * 3;
+#define BST(E, V)                                                                                                                         \
+  do {                                                                                                                                    \
+    static bool cfg = false;                                                                                                              \
+    if (!cfg) { cudaFuncSetAttribute(branches_step_kernel<E, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024); cfg = true; }  \
+    B200_LAUNCH((branches_step_kernel<E, V>), dim3((unsigned)T), dim3(kRowThreads), smem, (cudaStream_t)stream, x, init, y1, (const E*)w1, y2, \
+                (const E*)w2, y_scale, add, (const E*)step_vec, (const E*)norm_w, (E*)typed, (int)W, eps);                                \
+  } while (0)
+  const bool vec = W % 4 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(init) | reinterpret_cast<uintptr_t>(y1) |
+                                   reinterpret_cast<uintptr_t>(y2) | reinterpret_cast<uintptr_t>(add) | reinterpret_cast<uintptr_t>(typed)) & 15) == 0;
+  if (dt == B200_DT_F32) { if (vec) BST(float, 4); else BST(float, 1); }
+  else if (dt == B200_DT_BF16) { if (vec) BST(__nv_bfloat16, 4); else BST(__nv_bfloat16, 1); }
+  else { b200_set_last_error("unknown element type"); return B200_ERR_ARG; }
+#undef BST
+  b200_count_launches(1);
+  return B200_OK;
+}
+
+// in: rows of type in_dt (leading dimension ld_in), out: dense rows of type out_dt; act 0 SiLU, 1 GELU (tanh form), 2 tanh, 3 relu squared, 4 none
 extern "C" int b200_seq_ff_act(const void* in, int in_dt, int64_t ld_in, void* out, int out_dt, int64_t rows, int64_t F, int act, void* stream) {
   if (rows == 0 || F == 0) return B200_OK;
   int64_t blocks = (rows * F + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
-  if (act < 0 || act > 2) { b200_set_last_error("seq_ff_act: unknown activation"); return B200_ERR_ARG; }
+  if (act < 0 || act > 4) { b200_set_last_error("seq_ff_act: unknown activation"); return B200_ERR_ARG; }
 #define FA(TI, TO, A) B200_LAUNCH((ff_act_kernel<TI, TO, A>), dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, (const TI*)in, ld_in, (TO*)out, rows, (int)F)
 #define FA_ACT(TI, TO)            \
   do {                            \
     if (act == 0) FA(TI, TO, 0);  \
     else if (act == 1) FA(TI, TO, 1); \
-    else FA(TI, TO, 2);           \
+    else if (act == 2) FA(TI, TO, 2); \
+    else if (act == 3) FA(TI, TO, 3); \
+    else FA(TI, TO, 4);           \
   } while (0)
   if (in_dt == B200_DT_F32 && out_dt == B200_DT_F32) FA_ACT(float, float);
   else if (in_dt == B200_DT_F32 && out_dt == B200_DT_BF16) FA_ACT(float, __nv_bfloat16);

@@ -684,8 +684,7 @@ struct TalkPlan { int QT, KT; size_t smem; };
 static TalkPlan talk_mma_plan(int dt, int64_t T, int B, int H, int G, int d, int dv, bool has_talk) {
   static const bool use_mma = []() { const char* e = getenv("B200_SEQ_ATTN_MMA"); return !(e && e[0] == '0'); }();
   TalkPlan p{0, 0, 0};
-  if (!use_mma || dt != B200_DT_BF16 || G <= 0 || H % G != 0 || d % 16 != 0 || dv % 16 != 0 || dv > 128 || (dv / 8 != 2 && dv / 8 != 4 && dv / 8 != 8 && dv / 8 != 16))
-    return p;
+  if (!use_mma || dt != B200_DT_BF16 || G <= 0 || H % G != 0 || d % 16 != 0 || dv % 16 != 0 || dv > 128) return p;
   const int rep = H / G;
   int g16 = 16, x = rep;
   while (x % 2 == 0 && g16 > 1) { x /= 2; g16 /= 2; }   // g16 = 16 / gcd(16, rep)
@@ -759,7 +758,11 @@ extern "C" int b200_seq_talk_attn(const float* q, const void* cache, int dt, int
       switch (dv / 8) {
         case 2: TAM_KT(2); break;
         case 4: TAM_KT(4); break;
+        case 6: TAM_KT(6); break;
         case 8: TAM_KT(8); break;
+        case 10: TAM_KT(10); break;
+        case 12: TAM_KT(12); break;
+        case 14: TAM_KT(14); break;
         default: TAM_KT(16); break;
       }
 #undef TAM_KT

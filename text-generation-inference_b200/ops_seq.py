@@ -141,8 +141,8 @@ GATE_NONE, GATE_SILU_BEFORE, GATE_SIGMOID_AFTER, GATE_SILU_AFTER = 0, 1, 2, 3
 
 
 def group_rmsnorm_gate(x: torch.Tensor, weight: Optional[torch.Tensor], groups: int, eps: float, out_dtype: torch.dtype,
-                       gate: Optional[torch.Tensor] = None, gate_kind: int = GATE_NONE) -> torch.Tensor:
-    """x, gate: fp32 [T, C] column slices.  Per group of C / groups columns: v / sqrt(mean(v^2) + eps) * weight, with the gate
+                       gate: Optional[torch.Tensor] = None, gate_kind: int = GATE_NONE, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x, gate: fp32 [T, C] column slices (`out` may be one as well).  Per group of C / groups columns: v / sqrt(mean(v^2) + eps) * weight, with the gate
     multiplied in before the statistics (SiLU) or after the weight (sigmoid, or SiLU with GATE_SILU_AFTER).  groups == 0: no
     normalisation.  `weight` has one entry per column."""
     _cuda(x, weight, gate)
@@ -150,7 +150,9 @@ def group_rmsnorm_gate(x: torch.Tensor, weight: Optional[torch.Tensor], groups: 
     T, C = x.shape
     n = C // groups if groups > 0 else C
     assert groups == 0 or n * groups == C
-    out = torch.empty(T, C, dtype=out_dtype, device=x.device)
+    if out is None:
+        out = torch.empty(T, C, dtype=out_dtype, device=x.device)
+    assert out.dtype == out_dtype and out.shape == (T, C) and out.stride(1) == 1
     w_dt = _dt(weight) if weight is not None else _dt(out_dtype)
     _lib.check_seq(_lib.load_seq().b200_seq_group_rmsnorm_gate(
         _ptr(x), x.stride(0), _ptr(gate), gate.stride(0) if gate is not None else 0, gate_kind, _ptr(weight), w_dt, groups, n, float(eps),
@@ -454,17 +456,21 @@ def ff_gate(gate_up: torch.Tensor, act: int) -> torch.Tensor:
 
 
 def delta_scan(c: torch.Tensor, col_q: int, col_k: int, col_v: int, raw: torch.Tensor, col_b: int, col_a: int, A_log: torch.Tensor,
-               dt_bias: torch.Tensor, q_scale: float, S: torch.Tensor, step: RaggedStep, H: int, kv_heads: int, dk: int, dv: int) -> torch.Tensor:
+               dt_bias: torch.Tensor, q_scale: float, S: torch.Tensor, step: RaggedStep, H: int, kv_heads: int, dk: int, dv: int,
+               dec: Optional[torch.Tensor] = None, channels: bool = False) -> torch.Tensor:
     """Gated delta rule -> y fp32 [T, H * dv]; S fp32 [slots, H, dk, dv] advanced in place.  c fp32: activated q / k (kv_heads x dk
-    each) and v (H x dv) columns; raw fp32: write-strength logits at col_b and decay logits at col_a, one per head."""
-    _cuda(c, raw, S, A_log, dt_bias)
-    assert c.dtype == torch.float32 and raw.dtype == torch.float32 and S.dtype == torch.float32 and S.is_contiguous()
-    assert c.stride(1) == 1 and raw.stride(1) == 1 and A_log.dtype == dt_bias.dtype
+    each) and v (H x dv) columns; raw fp32: write-strength logits, one per head, at col_b; decay logits in `dec` (default: raw) from
+    col_a, one per head, or with `channels` one per head and key channel (H x dk; dt_bias alike): row n of S decays at rate n."""
+    dec = raw if dec is None else dec
+    _cuda(c, raw, dec, S, A_log, dt_bias)
+    assert c.dtype == torch.float32 and raw.dtype == torch.float32 and dec.dtype == torch.float32 and S.dtype == torch.float32 and S.is_contiguous()
+    assert c.stride(1) == 1 and raw.stride(1) == 1 and dec.stride(1) == 1 and A_log.dtype == dt_bias.dtype
+    assert A_log.numel() == H and dt_bias.numel() == (H * dk if channels else H)
     y = torch.empty(step.T, H * dv, dtype=torch.float32, device=c.device)
     _lib.check_seq(_lib.load_seq().b200_seq_delta_scan(
-        _ptr(c), c.stride(0), col_q, col_k, col_v, _ptr(raw), raw.stride(0), col_b, col_a, _ptr(A_log), _ptr(dt_bias), _dt(A_log), float(q_scale),
-        _ptr(S), _ptr(step.state_slots), _ptr(step.cu_q), _ptr(step.position_ids), _ptr(y), y.stride(0), step.B, H, kv_heads, dk, dv, _stream()),
-        "seq_delta_scan")
+        _ptr(c), c.stride(0), col_q, col_k, col_v, _ptr(raw), raw.stride(0), col_b, _ptr(dec), dec.stride(0), col_a, int(channels), _ptr(A_log),
+        _ptr(dt_bias), _dt(A_log), float(q_scale), _ptr(S), _ptr(step.state_slots), _ptr(step.cu_q), _ptr(step.position_ids), _ptr(y), y.stride(0),
+        step.B, H, kv_heads, dk, dv, _stream()), "seq_delta_scan")
     return y
 
 
@@ -533,12 +539,36 @@ def streams_step(X: torch.Tensor, *, init: Optional[torch.Tensor] = None, y: Opt
     return typed
 
 
-ACT_TANH = 2
+def branches_step(x: torch.Tensor, *, init: Optional[torch.Tensor] = None, branches=(), y_scale: float = 1.0, add: Optional[torch.Tensor] = None,
+                  step_vec: Optional[torch.Tensor] = None, norm_w: Optional[torch.Tensor] = None, eps: float = 0.0,
+                  dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
+    """One fp32 stream between two sublayers, x [T, W] in place (or started from `init`, then x is only written), in one launch:
+    x += y_scale * sum_i n(y_i) over up to two branches (y_i fp32 [T, W], w_i), n(y) = unit_rms(y) * w_i (w_i None: y itself); then
+    x += add (fp32 [T, W]) + step_vec [W]; returns unit_rms(x) * norm_w in norm_w's element type (norm_w None: nothing).  Weights and
+    step_vec share one element type (`dtype` when none of them is given)."""
+    ys, ws = [b[0] for b in branches] + [None] * (2 - len(branches)), [b[1] for b in branches] + [None] * (2 - len(branches))
+    _cuda(x, init, add, step_vec, norm_w, *ys, *ws)
+    assert len(branches) <= 2 and x.dtype == torch.float32 and x.is_contiguous() and x.dim() == 2
+    T, W = x.shape
+    for t in (init, add, *ys):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.shape == x.shape)
+    typed_args = [t for t in (*ws, step_vec, norm_w) if t is not None]
+    for t in typed_args:
+        assert t.dtype == typed_args[0].dtype and t.is_contiguous() and t.shape == (W,)
+    dt = typed_args[0].dtype if typed_args else (dtype or torch.float32)
+    typed = torch.empty(T, W, dtype=dt, device=x.device) if norm_w is not None else None
+    _lib.check_seq(_lib.load_seq().b200_seq_branches_step(_ptr(x), _ptr(init), _ptr(ys[0]), _ptr(ws[0]), _ptr(ys[1]), _ptr(ws[1]), float(y_scale),
+                                                          _ptr(add), _ptr(step_vec), _ptr(norm_w), _dt(dt), _ptr(typed), T, W, float(eps),
+                                                          _stream()), "seq_branches_step")
+    return typed
+
+
+ACT_TANH, ACT_RELU2, ACT_NONE = 2, 3, 4
 
 
 def ff_act(x: torch.Tensor, act: int, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
-    """act(x) element by element (ACT_SILU, ACT_GELU_TANH, ACT_TANH), evaluated in fp32; x [T, F] may be a column slice; fp32 rows may
-    come out in another element type."""
+    """act(x) element by element (ACT_SILU, ACT_GELU_TANH, ACT_TANH, ACT_RELU2: relu(x)^2, ACT_NONE: x itself), evaluated in fp32; x [T, F]
+    may be a column slice; fp32 rows may come out in another element type."""
     _cuda(x)
     assert x.dim() == 2 and x.stride(1) == 1
     out = torch.empty(x.shape, dtype=out_dtype or x.dtype, device=x.device)

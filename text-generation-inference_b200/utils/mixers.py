@@ -3,9 +3,10 @@ family can compose them: latent attention over a paged latent cache (sliding win
 scaling), the selective state-space mixer (Mamba-2 form), the matrix-memory mixer (mLSTM), differential attention (two soft-max
 maps per head, short convolutions after the projections, optionally over another layer's keys and values), attention with a
 learned bias per log-spaced distance bucket, the gated delta rule, attention with head-mixed scores under a chunked mask,
-windowed attention with sink logits, position-carrying values and a gate per head, the minimal gated recurrent unit, two mixers
-side by side on shared products, the generalised delta rule, and the feed-forward layers (clamped gated MLP, gated MLP with
-biases, plain MLP, routed experts with an optional shared expert).
+windowed or chunked attention with sink logits, position-carrying values and a gate per head, the minimal gated recurrent unit,
+the gated delta rule with a decay per key channel, two mixers side by side on shared products (their results added, or each normed
+first), the generalised delta rule, and the feed-forward layers (clamped gated MLP, gated MLP with biases, plain MLP, routed experts
+with an optional shared expert).
 
 A mixer declares what it keeps per sequence (`cache_spec`): a row of the paged cache per token, or fp32 state tensors in a
 state slot.  `forward(h, step, store)` takes the normed hidden states of a ragged step (ops_seq.RaggedStep: any mix of whole
@@ -465,14 +466,18 @@ class SinkRotaryAttention(nn.Module):
     and the whole k projection (a weight per column), rotation of the first `rotary.dims` columns of every q / k head (column i
     with column i + dims / 2).  Cached per token: rotated keys and turned values of all key heads (token-major row); per
     sequence: the last conv - 1 projected rows (fp32).
+    Every part but the soft-max is optional: `sink`, `head_gate`, `qk_norm` False and `rotary` / `value_rotary` None leave theirs out,
+    `bias` adds q.b / k.b / v.b to the projections, `window` (the last so many keys) and `chunk` (keys of the query's own chunk of so
+    many positions, counted from position 0) are the masks.
     A mixer that can share its input and output products with a neighbour: `in_rows()` are the rows it adds to the input
-    projection, `from_projection` continues from the fp32 projection and leaves the gated heads, times `out_scale`, in `out`;
-    `w_o` finishes.
-    Tensors under `prefix`: q, k, v, [q.conv, k.conv, v.conv,] q.norm, k.norm, [sink,] [g,] o."""
+    projection (`in_bias()` their biases), `from_projection` continues from the fp32 projection and leaves the gated heads, times
+    `out_scale`, in `out`; `w_o` finishes.
+    Tensors under `prefix`: q, k, v, [q.b, k.b, v.b,] [q.conv, k.conv, v.conv,] [q.norm, k.norm,] [sink,] [g,] o."""
 
     def __init__(self, prefix: str, weights, *, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, rotary: Optional[ScaledRotaryTables],
                  value_rotary: Optional[ScaledRotaryTables], value_pairs: str = "halves", conv: int = 0, window: Optional[int] = None,
-                 sink: bool = True, head_gate: bool = True, eps: float = 1e-6):
+                 sink: bool = True, head_gate: bool = True, eps: float = 1e-6, qk_norm: bool = True, bias: bool = False,
+                 chunk: Optional[int] = None):
         super().__init__()
         _need_single_rank(weights, "SinkRotaryAttention")
         if heads % kv_heads:
@@ -481,6 +486,7 @@ class SinkRotaryAttention(nn.Module):
             raise ValueError("value_pairs is 'halves' or 'interleaved'")
         self.H, self.G, self.d, self.dv, self.taps = int(heads), int(kv_heads), int(dim), int(vdim), int(conv or 0)
         self.scale, self.rotary, self.value_rotary, self.window, self.eps = float(scale), rotary, value_rotary, int(window or 0), float(eps)
+        self.chunk = int(chunk or 0)
         self.value_interleaved = value_pairs == "interleaved"
         if rotary is not None and rotary.dims > dim:
             raise ValueError("rotary dims exceed the head size")
@@ -492,18 +498,27 @@ class SinkRotaryAttention(nn.Module):
         self.w_in = torch.cat([get(n) for n in (("q", "k", "v", "g") if head_gate else ("q", "k", "v"))], 0).contiguous()
         self.n_in = self.channels + (self.H if head_gate else 0)
         self.head_gate = bool(head_gate)
+        self.b_in = None
+        if bias:   # the gate has none: zeros, so that the products can run as one
+            parts = [get(f"{n}.b") for n in ("q", "k", "v")]
+            self.b_in = torch.cat(parts + ([parts[0].new_zeros(self.H)] if head_gate else []), 0).contiguous()
         self.conv_w = torch.cat([get(f"{n}.conv") for n in ("q", "k", "v")], 0).contiguous() if self.taps >= 1 else None
-        self.q_norm, self.k_norm = get("q.norm").contiguous(), get("k.norm").contiguous()
+        self.qk_norm = bool(qk_norm)
+        self.q_norm, self.k_norm = (get("q.norm").contiguous(), get("k.norm").contiguous()) if qk_norm else (None, None)
         self.sink = get("sink").float().contiguous() if sink else None
         self.w_o = get("o").contiguous()
         self.dtype = self.w_o.dtype
         self.n_out = self.H * self.dv
         if self.w_in.shape[0] != self.n_in or (self.conv_w is not None and self.conv_w.shape != (self.channels, self.taps)) or \
-                self.w_o.shape[1] != self.n_out or (self.sink is not None and self.sink.shape != (self.H,)):
+                self.w_o.shape[1] != self.n_out or (self.sink is not None and self.sink.shape != (self.H,)) or \
+                (self.b_in is not None and self.b_in.shape != (self.n_in,)):
             raise ValueError(f"{prefix}: tensor shapes do not match the head sizes")
 
     def in_rows(self) -> torch.Tensor:
         return self.w_in
+
+    def in_bias(self) -> Optional[torch.Tensor]:
+        return self.b_in
 
     def cache_spec(self) -> LayerCacheSpec:
         state = {"conv": (max(self.taps - 1, 1), self.channels)} if self.taps >= 1 else {}   # a single tap is a weight per channel
@@ -524,18 +539,18 @@ class SinkRotaryAttention(nn.Module):
         vr = self.value_rotary
         vcos, vsin = vr.tables(max_s, u.device) if vr is not None else (None, None)
         q = ops.qk_rot_prepare(c, col_q=cq, col_k=cq + self.cq, col_v=cq + self.cq + self.ck, heads=self.H, kv_heads=self.G, dim=self.d,
-                               vdim=self.dv, q_norm_w=self.q_norm, k_norm_w=self.k_norm, whole_norm=True, eps=self.eps, cos=cos, sin=sin,
+                               vdim=self.dv, q_norm_w=self.q_norm, k_norm_w=self.k_norm, whole_norm=self.qk_norm, eps=self.eps, cos=cos, sin=sin,
                                rot=self.rotary.dims if self.rotary is not None else 0, step=step, cache=pages, k_off=0, v_off=self.ck,
                                v_cos=vcos, v_sin=vsin, v_rot=vr.dims if vr is not None else 0, v_interleaved=self.value_interleaved)
-        a = ops.talk_attn(q, pages, step, kv_heads=self.G, vdim=self.dv, k_off=0, v_off=self.ck, scale=self.scale, window=self.window,
-                          sink=self.sink)
+        a = ops.talk_attn(q, pages, step, kv_heads=self.G, vdim=self.dv, k_off=0, v_off=self.ck, scale=self.scale, chunk=self.chunk,
+                          window=self.window, sink=self.sink)
         gate = u[:, col0 + self.channels:col0 + self.channels + self.H] if self.head_gate else None
         ops.heads_turn_gate(a, gate, vcos, vsin, vr.dims if vr is not None else 0, self.value_interleaved, step, self.dtype, out=out,
                             out_scale=out_scale)
 
     def forward(self, h: torch.Tensor, step: ops.RaggedStep, pages: torch.Tensor, state, max_s: int) -> torch.Tensor:
         """-> fp32 [T, width]"""
-        u = ops.linear(h, self.w_in, out_dtype=torch.float32)
+        u = ops.linear(h, self.w_in, self.b_in, out_dtype=torch.float32)
         o = torch.empty(step.T, self.n_out, dtype=self.dtype, device=h.device)
         self.from_projection(u, 0, step, pages, state, max_s, o)
         return ops.linear(o, self.w_o, out_dtype=torch.float32)
@@ -579,6 +594,86 @@ class MinGRUMixer(nn.Module):
         return ops.linear(o, self.w_o, out_dtype=torch.float32)
 
 
+class ChannelDeltaMixer(nn.Module):
+    """Gated delta rule whose memory rows decay each at their own rate: as `GatedDeltaMixer` (convolutions + SiLU on q / k / v, unit-length
+    q and k, S <- diag(g) S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q), with one decay per head and key channel from a low-rank
+    projection, g = exp(-exp(A_log_head) softplus(W_a2 W_a1 h + dt_bias)), and an output gate from another one: each head's o is
+    divided by its RMS, times a weight shared by the heads, times sigmoid(W_g2 W_g1 h).  State per sequence: S and the last
+    conv - 1 convolution inputs, both fp32.  Shares products with a neighbour like `SinkRotaryAttention`.
+    The two low-rank products run as one: W_a1 and W_g1 are rows of the input projection (padded with zero rows to a rank that the
+    tensor-core product takes), and [W_a2 0; 0 W_g2] maps that latent to [decay logits | gate logits] - the zeros add nothing.
+    Tensors under `prefix`: q, q.conv, k, k.conv, v, v.conv, b, A_log, a1, a2, dt_bias, g1, g2, norm, o."""
+
+    def __init__(self, prefix: str, weights, *, heads: int, kv_heads: int, dim: int, vdim: int, conv: int, eps: float):
+        super().__init__()
+        _need_single_rank(weights, "ChannelDeltaMixer")
+        if heads % kv_heads:
+            raise ValueError("heads must be a multiple of kv_heads")
+        self.H, self.G, self.d, self.dv, self.taps, self.eps = int(heads), int(kv_heads), int(dim), int(vdim), int(conv), float(eps)
+        get = lambda n: weights.get_tensor(f"{prefix}.{n}")  # noqa: E731
+        self.cqk, self.n, self.n_out = self.G * self.d, self.H * self.d, self.H * self.dv
+        self.channels = 2 * self.cqk + self.n_out                                         # convolved columns [q | k | v]
+        a1, g1, a2, g2 = get("a1"), get("g1"), get("a2"), get("g2")
+        ra, rg = a1.shape[0], g1.shape[0]
+        self.rank = max(64, (ra + rg + 7) // 8 * 8)
+        pad = a1.new_zeros(self.rank - ra - rg, a1.shape[1])
+        self.w_in = torch.cat([get("q"), get("k"), get("v"), a1, g1, pad, get("b")], 0).contiguous()   # -> [q | k | v | latent | beta]
+        self.n_in = self.channels + self.rank + self.H
+        self.conv_w = torch.cat([get(f"{n}.conv") for n in ("q", "k", "v")], 0).contiguous()
+        self.A_log, self.dt_bias = get("A_log").contiguous(), get("dt_bias").contiguous()
+        self.norm_w = get("norm").repeat(self.H).contiguous()                             # one entry per column of the heads
+        self.w_o = get("o").contiguous()
+        self.dtype = self.w_o.dtype
+        if self.w_in.shape[0] != self.n_in or self.conv_w.shape != (self.channels, self.taps) or a2.shape != (self.n, ra) or \
+                g2.shape != (self.n_out, rg) or self.dt_bias.shape != (self.n,) or self.A_log.shape != (self.H,) or \
+                self.norm_w.shape != (self.n_out,) or self.w_o.shape[1] != self.n_out:
+            raise ValueError(f"{prefix}: tensor shapes do not match the head sizes")
+        self.w_low = a2.new_zeros(self.n + self.n_out, self.rank)
+        self.w_low[:self.n, :ra] = a2
+        self.w_low[self.n:, ra:ra + rg] = g2
+
+    def in_rows(self) -> torch.Tensor:
+        return self.w_in
+
+    def in_bias(self) -> Optional[torch.Tensor]:
+        return None
+
+    def cache_spec(self) -> LayerCacheSpec:
+        return LayerCacheSpec(kind="state", state={"S": (self.H, self.d, self.dv), "conv": (max(self.taps - 1, 1), self.channels)})
+
+    def from_projection(self, u: torch.Tensor, col0: int, step: ops.RaggedStep, pages, state, max_s: int, out: torch.Tensor,
+                        out_scale: float = 1.0) -> None:
+        """u fp32 [T, >= col0 + n_in]: this mixer's input projection from column col0 -> out [T, heads * vdim] (a column slice is fine)"""
+        if out_scale != 1.0:
+            raise NotImplementedError("ChannelDeltaMixer: the result is not scaled before its output projection")
+        C, R = self.channels, self.rank
+        low = ops.linear(ops.ff_act(u[:, col0 + C:col0 + C + R], ops.ACT_NONE, out_dtype=self.dtype), self.w_low, out_dtype=torch.float32)
+        c = ops.causal_conv(u, col0, C, self.conv_w, None, state["conv"], step, act_silu=True)
+        y = ops.delta_scan(c, 0, self.cqk, 2 * self.cqk, u, col0 + C + R, 0, self.A_log, self.dt_bias, self.d ** -0.5, state["S"], step,
+                           self.H, self.G, self.d, self.dv, dec=low, channels=True)
+        ops.group_rmsnorm_gate(y, self.norm_w, self.H, self.eps, self.dtype, gate=low[:, self.n:], gate_kind=ops.GATE_SIGMOID_AFTER, out=out)
+
+    def forward(self, h: torch.Tensor, step: ops.RaggedStep, pages, state: Dict[str, torch.Tensor], max_s: int) -> torch.Tensor:
+        """-> fp32 [T, width]"""
+        u = ops.linear(h, self.w_in, out_dtype=torch.float32)
+        o = torch.empty(step.T, self.n_out, dtype=self.dtype, device=h.device)
+        self.from_projection(u, 0, step, pages, state, max_s, o)
+        return ops.linear(o, self.w_o, out_dtype=torch.float32)
+
+
+def _side_by_side_spec(left: nn.Module, right: nn.Module) -> LayerCacheSpec:
+    """what a layer with both mixers keeps: at most one of them paged rows, the state tensors of both under `left.` / `right.` names"""
+    sl, sr = left.cache_spec(), right.cache_spec()
+    if sl.kind == "paged" and sr.kind == "paged":
+        raise NotImplementedError("two paged mixers in one layer")
+    return LayerCacheSpec(kind="paged" if "paged" in (sl.kind, sr.kind) else "state", row_width=max(sl.row_width, sr.row_width),
+                          state={**{f"left.{k}": v for k, v in (sl.state or {}).items()}, **{f"right.{k}": v for k, v in (sr.state or {}).items()}})
+
+
+def _side_state(state: Optional[Dict[str, torch.Tensor]], prefix: str) -> Dict[str, torch.Tensor]:
+    return {k[len(prefix):]: v for k, v in (state or {}).items() if k.startswith(prefix)}
+
+
 class ParallelMixers(nn.Module):
     """Two mixers side by side that read the same input: left_scale * left(h) + right_scale * right(h).  Both must offer
     `in_rows` / `from_projection` / `w_o` / `n_in` / `n_out`: their input projections run as ONE product, each leaves what its
@@ -592,12 +687,7 @@ class ParallelMixers(nn.Module):
         self.w_in = torch.cat([left.in_rows(), right.in_rows()], 0).contiguous()
         self.w_o = torch.cat([left.w_o, right.w_o], 1).contiguous()
         self.dtype = self.w_o.dtype
-        sl, sr = left.cache_spec(), right.cache_spec()
-        if sl.kind == "paged" and sr.kind == "paged":
-            raise NotImplementedError("two paged mixers in one layer")
-        self._spec = LayerCacheSpec(kind="paged" if "paged" in (sl.kind, sr.kind) else "state", row_width=max(sl.row_width, sr.row_width),
-                                    state={**{f"left.{k}": v for k, v in (sl.state or {}).items()},
-                                           **{f"right.{k}": v for k, v in (sr.state or {}).items()}})
+        self._spec = _side_by_side_spec(left, right)
 
     def cache_spec(self) -> LayerCacheSpec:
         return self._spec
@@ -612,10 +702,50 @@ class ParallelMixers(nn.Module):
         L, R = self.left, self.right
         u = ops.linear(h, self.w_in, out_dtype=torch.float32)
         o = torch.empty(step.T, L.n_out + R.n_out, dtype=self.dtype, device=h.device)
-        side = lambda p: {k[len(p):]: v for k, v in (state or {}).items() if k.startswith(p)}  # noqa: E731
-        L.from_projection(u, 0, step, pages, side("left."), max_s, o[:, :L.n_out], self.ls)
-        R.from_projection(u, L.n_in, step, pages, side("right."), max_s, o[:, L.n_out:], self.rs)
+        L.from_projection(u, 0, step, pages, _side_state(state, "left."), max_s, o[:, :L.n_out], self.ls)
+        R.from_projection(u, L.n_in, step, pages, _side_state(state, "right."), max_s, o[:, L.n_out:], self.rs)
         return ops.linear(o, self.w_o, out_dtype=torch.float32)
+
+
+class NormedParallelMixers(nn.Module):
+    """Two mixers side by side that read the same input and whose results are normed before they are added:
+    out_scale * (unit_rms(left(h)) * w_left + unit_rms(right(h)) * w_right).  Both must offer `in_rows` / `in_bias` / `from_projection` /
+    `w_o` / `n_in` / `n_out`; their input projections run as ONE product.  `forward` returns the two results before their norms with
+    the norm weights, [(fp32 [T, width], weight), ...]: norms, scale and sum belong to the launch that writes the residual stream
+    (ops.branches_step with y_scale = `out_scale`).  Stores as in `ParallelMixers`.
+    Tensors under `prefix`: left.out, right.out (besides the mixers' own)."""
+
+    def __init__(self, prefix: str, weights, left: nn.Module, right: nn.Module, out_scale: float = 0.5):
+        super().__init__()
+        self.left, self.right, self.out_scale = left, right, float(out_scale)
+        self.w_in = torch.cat([left.in_rows(), right.in_rows()], 0).contiguous()
+        biases = [left.in_bias(), right.in_bias()]
+        self.b_in = None
+        if any(b is not None for b in biases):
+            self.b_in = torch.cat([self.w_in.new_zeros(m.n_in) if b is None else b for m, b in zip((left, right), biases)], 0).contiguous()
+        self.norm_left, self.norm_right = weights.get_tensor(f"{prefix}.left.out").contiguous(), weights.get_tensor(f"{prefix}.right.out").contiguous()
+        self.dtype = self.w_in.dtype
+        self._spec = _side_by_side_spec(left, right)
+        left.w_in = right.w_in = left.b_in = None    # the joined product owns the rows
+
+    def cache_spec(self) -> LayerCacheSpec:
+        return self._spec
+
+    def prepare_positions(self, n_pos: int, device) -> None:
+        for m in (self.left, self.right):
+            if hasattr(m, "prepare_positions"):
+                m.prepare_positions(n_pos, device)
+
+    def forward(self, h: torch.Tensor, step: ops.RaggedStep, pages, state: Dict[str, torch.Tensor], max_s: int) -> list:
+        L, R = self.left, self.right
+        u = ops.linear(h, self.w_in, self.b_in, out_dtype=torch.float32)
+        ol = torch.empty(step.T, L.n_out, dtype=self.dtype, device=h.device)
+        L.from_projection(u, 0, step, pages, _side_state(state, "left."), max_s, ol)
+        left = ops.linear(ol, L.w_o, out_dtype=torch.float32)
+        orr = torch.empty(step.T, R.n_out, dtype=self.dtype, device=h.device)
+        R.from_projection(u, L.n_in, step, pages, _side_state(state, "right."), max_s, orr)
+        right = ops.linear(orr, R.w_o, out_dtype=torch.float32)
+        return [(left, self.norm_left), (right, self.norm_right)]
 
 
 class GeneralDeltaMixer(nn.Module):
@@ -656,17 +786,20 @@ class GeneralDeltaMixer(nn.Module):
 
 
 class PlainMLP(nn.Module):
-    """down(act(up x)) with act SiLU or the tanh form of GELU, no gate, no biases.  The result is fp32.
-    Tensors under `prefix`: up, down."""
+    """down(act(up x [+ b_up])) [+ b_down] with act SiLU, the tanh form of GELU or the square of ReLU, no gate.  The result is fp32.
+    Tensors under `prefix`: up, down [, up.b, down.b]."""
 
-    def __init__(self, prefix: str, weights, *, activation: str):
+    _ACTS = {"silu": ops.ACT_SILU, "gelu_tanh": ops.ACT_GELU_TANH, "relu2": ops.ACT_RELU2}
+
+    def __init__(self, prefix: str, weights, *, activation: str, bias: bool = False):
         super().__init__()
         _need_single_rank(weights, "PlainMLP")
-        if activation not in ("silu", "gelu_tanh"):
+        if activation not in self._ACTS:
             raise NotImplementedError(f"activation {activation!r}")
-        self.act = ops.ACT_SILU if activation == "silu" else ops.ACT_GELU_TANH
+        self.act = self._ACTS[activation]
         self.w_up = weights.get_tensor(f"{prefix}.up").contiguous()
         self.w_down = weights.get_tensor(f"{prefix}.down").contiguous()
+        self.b_up, self.b_down = (weights.get_tensor(f"{prefix}.{n}.b").contiguous() if bias else None for n in ("up", "down"))
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
-        return ops.linear(ops.ff_act(ops.linear(h, self.w_up), self.act), self.w_down, out_dtype=torch.float32)
+        return ops.linear(ops.ff_act(ops.linear(h, self.w_up, self.b_up), self.act), self.w_down, self.b_down, out_dtype=torch.float32)
