@@ -1142,7 +1142,7 @@ def _stream_family_measure(raw, cfg, op_names, PB, PL, DB, DL, K, Wm, timed, lib
 
 
 def _noganex_side(width, env):
-    """the Noganex half of --noganex-compare (also the partner of --nasozen-compare) -> its result entry"""
+    """the Noganex half of --noganex-compare (also the partner of --nasozen-compare and --nomalorn-compare) -> its result entry"""
     from tgis_b200.models.custom_modeling import noganex_modeling
     from tgis_b200.utils.synthetic import noganex_config
     PB, PL, DB, DL, K, Wm, ctx = (env[k] for k in ("PB", "PL", "DB", "DL", "K", "Wm", "ctx"))
@@ -1180,31 +1180,21 @@ def _noganex_side(width, env):
     return common(f"noganex-w{width}", raw, r, kernels, {"experts": moes[0]["router"]["experts"], "top": top})
 
 
-def run_noganex_compare(args):
-    """Noganex (bfloat16) beside Dubesun (bfloat16), the closest family of the engine (fp32 stream, attention over a paged cache, short
-    convolutions, routed experts), at equal width and depth on random weights: prefill of 4 x 1024 tokens and decode of 32 sequences at
-    context 1024, measured as --dubesun-compare measures its pair, with the achieved FLOP/s or bytes/s of the kernels that carry a step
-    against the measured peaks."""
+def _stream_compare_env(args):
+    """what the comparisons of the fp32-stream families share: shapes of the timed steps, measured peaks, the L2-flushing timer and the
+    layout of a result entry"""
     import torch
-    import tgis_b200  # noqa: F401
     from tgis_b200 import _lib as _libmod
-    from tgis_b200.models.custom_modeling import dubesun_modeling
-    from tgis_b200.utils.synthetic import dubesun_config
-
     pk = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
     if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")):
         with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
             d = json.load(f)
         pk = {"hbm_gbs": float(d["hbm_gbs"]), "bf16_tflops": float(d["bf16_tflops"]), "source": "measured"}
-    hbm, tens = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
     dev = torch.device("cuda", 0)
     torch.cuda.set_device(dev)
     flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
     PB, PL, DB, DL = 4, 1024, 32, 1024
     K, Wm = max(args.steps // 4, 4), args.warmup
-    ctx = DL + Wm + K + 2
-    lib = _libmod.load_seq()
-    results = []
 
     def timed(fn, n):
         total = 0.0
@@ -1232,9 +1222,30 @@ def run_noganex_compare(args):
     def us(dec_k, *prefixes):
         return sum(v for k, v in dec_k.items() if k.startswith(prefixes))
 
-    widths = (2048, 4096) if not args.layers else (2048,)
-    env = dict(PB=PB, PL=PL, DB=DB, DL=DL, K=K, Wm=Wm, ctx=ctx, timed=timed, lib=lib, hbm=hbm, tens=tens, common=common, us=us)
-    for width in widths:
+    def report(metric, results):
+        print(json.dumps({"metric": metric, "unit": "tokens/s", "n_gpus": 1, "steps": K, "warmup": Wm, "data": "synthetic",
+                          "config": {"prefill": [PB, PL], "decode": [DB, DL], "l2": "flushed between timed calls"},
+                          "peaks": {"hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"], "source": pk.get("source")}, "models": results}))
+        return 0
+
+    return dict(PB=PB, PL=PL, DB=DB, DL=DL, K=K, Wm=Wm, ctx=DL + Wm + K + 2, timed=timed, lib=_libmod.load_seq(), hbm=pk["hbm_gbs"] * 1e9,
+                tens=pk["bf16_tflops"] * 1e12, common=common, us=us, report=report, widths=(2048, 4096) if not args.layers else (2048,))
+
+
+def run_noganex_compare(args):
+    """Noganex (bfloat16) beside Dubesun (bfloat16), the closest family of the engine (fp32 stream, attention over a paged cache, short
+    convolutions, routed experts), at equal width and depth on random weights: prefill of 4 x 1024 tokens and decode of 32 sequences at
+    context 1024, measured as --dubesun-compare measures its pair, with the achieved FLOP/s or bytes/s of the kernels that carry a step
+    against the measured peaks."""
+    import tgis_b200  # noqa: F401
+    from tgis_b200.models.custom_modeling import dubesun_modeling
+    from tgis_b200.utils.synthetic import dubesun_config
+
+    env = _stream_compare_env(args)
+    PB, PL, DB, DL, K, Wm, ctx = (env[k] for k in ("PB", "PL", "DB", "DL", "K", "Wm", "ctx"))
+    timed, lib, hbm, tens, common, us = (env[k] for k in ("timed", "lib", "hbm", "tens", "common", "us"))
+    results = []
+    for width in env["widths"]:
         results.append(_noganex_side(width, env))
         # ---------------------------------------------------------------- Dubesun, the partner
         raw = dubesun_config(f"dubesun-w{width}")
@@ -1266,10 +1277,7 @@ def run_noganex_compare(args):
             "linear decode (tcgen05 projections)": {"us": g_us, "of_measured_hbm": (proj_w + head_w) * 2 / (max(g_us, 1e-9) * 1e-6) / hbm},
         }
         results.append(common(f"dubesun-w{width}", raw, r, kernels, {"experts": f["router"]["experts"], "top": top}))
-    print(json.dumps({"metric": "noganex_compare", "unit": "tokens/s", "n_gpus": 1, "steps": K, "warmup": Wm, "data": "synthetic",
-                      "config": {"prefill": [PB, PL], "decode": [DB, DL], "l2": "flushed between timed calls"},
-                      "peaks": {"hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"], "source": pk.get("source")}, "models": results}))
-    return 0
+    return env["report"]("noganex_compare", results)
 
 
 def run_nasozen_compare(args):
@@ -1277,56 +1285,15 @@ def run_nasozen_compare(args):
     rotate-half rotation in front of the same attention kernel, a delta-rule memory, routed experts), at equal width and depth on random
     weights: prefill of 4 x 1024 tokens and decode of 32 sequences at context 1024, measured as --noganex-compare measures its pair, with
     the achieved FLOP/s or bytes/s of the kernels that carry a step against the measured peaks."""
-    import torch
     import tgis_b200  # noqa: F401
-    from tgis_b200 import _lib as _libmod
     from tgis_b200.models.custom_modeling import nasozen_modeling
     from tgis_b200.utils.synthetic import nasozen_config
 
-    pk = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
-    if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")):
-        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
-            d = json.load(f)
-        pk = {"hbm_gbs": float(d["hbm_gbs"]), "bf16_tflops": float(d["bf16_tflops"]), "source": "measured"}
-    hbm, tens = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
-    dev = torch.device("cuda", 0)
-    torch.cuda.set_device(dev)
-    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
-    PB, PL, DB, DL = 4, 1024, 32, 1024
-    K, Wm = max(args.steps // 4, 4), args.warmup
-    ctx = DL + Wm + K + 2
-    lib = _libmod.load_seq()
+    env = _stream_compare_env(args)
+    PB, PL, DB, DL, K, Wm, ctx = (env[k] for k in ("PB", "PL", "DB", "DL", "K", "Wm", "ctx"))
+    timed, lib, hbm, tens, common, us = (env[k] for k in ("timed", "lib", "hbm", "tens", "common", "us"))
     results = []
-
-    def timed(fn, n):
-        total = 0.0
-        for _ in range(n):
-            flush.zero_()
-            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            e0.record()
-            fn()
-            e1.record()
-            torch.cuda.synchronize()
-            total += e0.elapsed_time(e1)
-        return total / n
-
-    def common(name, raw, r, kernels, extra):
-        out = {"model": name, "dtype": "bf16", "layers": len(raw["layers"]), "prefill_tokens_per_s": PB * PL / (r["pre_ms"] * 1e-3),
-               "decode_tokens_per_s": DB / (r["dec_ms"] * 1e-3), "prefill_ms": r["pre_ms"], "decode_ms_per_step": r["dec_ms"],
-               "decode_graph_tokens_per_s": DB / (r["graph_ms"] * 1e-3), "decode_graph_ms_per_step": r["graph_ms"],
-               "prefill_ms_by_op": {k: round(v, 4) for k, v in r["pre_ops"].items()},
-               "decode_ms_by_op": {k: round(v, 4) for k, v in r["dec_ops"].items()},
-               "decode_graph_us_by_kernel": {k: round(v, 2) for k, v in sorted(r["dec_k"].items(), key=lambda kv: -kv[1])},
-               "decode_graph_traced_us": r["dec_total"], "kernels": kernels}
-        out.update(extra)
-        return out
-
-    def us(dec_k, *prefixes):
-        return sum(v for k, v in dec_k.items() if k.startswith(prefixes))
-
-    env = dict(PB=PB, PL=PL, DB=DB, DL=DL, K=K, Wm=Wm, ctx=ctx, timed=timed, lib=lib, hbm=hbm, tens=tens, common=common, us=us)
-    widths = (2048, 4096) if not args.layers else (2048,)
-    for width in widths:
+    for width in env["widths"]:
         raw = nasozen_config(f"nasozen-w{width}")
         names = ["linear", "embed_scale", "streams_step", "causal_conv", "qk_rot_prepare", "talk_attn", "heads_turn_gate", "mingru_scan", "mlstm_scan",
                  "gdelta_scan", "group_rmsnorm_gate", "ff_act", "moe_route", "moe_gather_rows", "moe_linear", "ff_gate", "moe_combine_add"]
@@ -1376,10 +1343,61 @@ def run_nasozen_compare(args):
         }
         results.append(common(f"nasozen-w{width}", raw, r, kernels, {"experts": moes[0]["router"]["experts"], "top": top, "streams": S}))
         results.append(_noganex_side(width, env))
-    print(json.dumps({"metric": "nasozen_compare", "unit": "tokens/s", "n_gpus": 1, "steps": K, "warmup": Wm, "data": "synthetic",
-                      "config": {"prefill": [PB, PL], "decode": [DB, DL], "l2": "flushed between timed calls"},
-                      "peaks": {"hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"], "source": pk.get("source")}, "models": results}))
-    return 0
+    return env["report"]("nasozen_compare", results)
+
+
+def run_nomalorn_compare(args):
+    """Nomalorn (bfloat16) beside Noganex (bfloat16), the closest family of the engine (the gated delta rule behind short convolutions,
+    chunked grouped-query attention with partly rotated heads, an fp32 stream), at equal width and number of layer runs on random
+    weights: prefill of 4 x 1024 tokens and decode of 32 sequences at context 1024, measured as --noganex-compare measures its pair,
+    with the achieved FLOP/s or bytes/s of the kernels that carry a step against the measured peaks."""
+    import tgis_b200  # noqa: F401
+    from tgis_b200.models.custom_modeling import nomalorn_modeling
+    from tgis_b200.utils.synthetic import nomalorn_config
+
+    env = _stream_compare_env(args)
+    PB, PL, DB, DL, K, Wm, ctx = (env[k] for k in ("PB", "PL", "DB", "DL", "K", "Wm", "ctx"))
+    timed, lib, hbm, tens, common, us = (env[k] for k in ("timed", "lib", "hbm", "tens", "common", "us"))
+    results = []
+    for width in env["widths"]:
+        raw = nomalorn_config(f"nomalorn-w{width}")
+        names = ["linear", "embed_scale", "branches_step", "causal_conv", "qk_rot_prepare", "talk_attn", "heads_turn_gate", "delta_scan",
+                 "group_rmsnorm_gate", "ff_act", "rmsnorm_rows"]
+        cfg = nomalorn_modeling.NomalornConfig(raw)
+        r = _stream_family_measure(raw, cfg, names, PB, PL, DB, DL, K, Wm, timed, lib)
+        shapes = nomalorn_modeling.tensor_shapes(raw)
+        runs = [raw["layers"][i] for i, _ in cfg.layer_runs]
+        left, right, T = [l["mixer"]["left"] for l in runs], [l["mixer"]["right"] for l in runs], PB * PL
+        attn_flops = sum(PB * (PL * (PL + 1) // 2) * m["heads"] * (m["dim"] + m["vdim"]) * 2 for m in left)
+        attn_row = sum(m["kv_heads"] * (m["dim"] + m["vdim"]) for m in left)       # elements a decoding token reads per cached token
+        state_b = sum(m["heads"] * m["dim"] * m["vdim"] * 4 * 2 for m in right)    # state read + written per sequence and step
+        # one multiply by the decay and three multiply-adds (prediction, write, read-out) per state entry and token
+        scan_flops = sum(T * m["heads"] * m["dim"] * m["vdim"] * 7 for m in right)
+        scan_in = sum((m["kv_heads"] * m["dim"] * 2 + m["heads"] * (m["dim"] + 2 * m["vdim"])) * 4 for m in right)   # fp32 rows in and out per token
+        # the stream in and out at every boundary, two branches (mixer) or one (feed-forward) in, the typed copy out
+        stream_b = sum(width * ((8 + 8 + 2) + ((8 + 4 + 2) if l["mlp"] else 0)) for l in runs) + width * (4 + 4 + 2)
+        run_w = [sum(a * b for n, (a, *rest) in shapes.items() for b in rest[:1] if n.startswith(f"l{i}.")) for i, _ in cfg.layer_runs]
+        dense_w, head_w = sum(run_w), shapes["embed"][0] * shapes["embed"][1]
+        lin_flops = 2 * T * dense_w + 2 * PB * head_w
+        pre, dk = r["pre_ops"], r["dec_k"]
+        a_us, s_us, g_us, b_us = us(dk, "talk_attn"), us(dk, "delta_scan"), dk.get("gemm_f16_kernel", 0.0), us(dk, "branches_step")
+        kernels = {
+            "talk_attn prefill": {"ms": pre["talk_attn"], "tflops": attn_flops / pre["talk_attn"] / 1e9,
+                                  "of_measured_tensor": attn_flops / (pre["talk_attn"] * 1e-3) / tens},
+            "talk_attn decode": {"us": a_us, "of_measured_hbm": DB * ctx * attn_row * 2 / (max(a_us, 1e-9) * 1e-6) / hbm},
+            "delta_scan prefill": {"ms": pre["delta_scan"], "tokens_per_s_per_layer": T * len(right) / (pre["delta_scan"] * 1e-3),
+                                   "fp32_tflops": scan_flops / pre["delta_scan"] / 1e9,
+                                   "of_measured_hbm": (T * scan_in + PB * state_b / 2) / (pre["delta_scan"] * 1e-3) / hbm},
+            "delta_scan decode": {"us": s_us, "of_measured_hbm": DB * state_b / (max(s_us, 1e-9) * 1e-6) / hbm},
+            "branches_step prefill": {"ms": pre["branches_step"], "of_measured_hbm": T * stream_b / (pre["branches_step"] * 1e-3) / hbm},
+            "branches_step decode": {"us": b_us, "launches": 1 + sum(2 if l["mlp"] else 1 for l in runs),
+                                     "of_measured_hbm": DB * stream_b / (max(b_us, 1e-9) * 1e-6) / hbm},
+            "linear prefill": {"ms": pre["linear"], "of_measured_tensor": lin_flops / (pre["linear"] * 1e-3) / tens},
+            "linear decode (tcgen05 projections)": {"us": g_us, "of_measured_hbm": (dense_w + head_w) * 2 / (max(g_us, 1e-9) * 1e-6) / hbm},
+        }
+        results.append(common(f"nomalorn-w{width}", raw, r, kernels, {"layer_runs": len(runs)}))
+        results.append(_noganex_side(width, env))
+    return env["report"]("nomalorn_compare", results)
 
 
 def main():
@@ -1402,6 +1420,8 @@ def main():
                     help="Noganex beside Dubesun at equal size: prefill and decode throughput and per-kernel rooflines (one GPU)")
     ap.add_argument("--nasozen-compare", action="store_true",
                     help="Nasozen beside Noganex at equal size: prefill and decode throughput and per-kernel rooflines (one GPU)")
+    ap.add_argument("--nomalorn-compare", action="store_true",
+                    help="Nomalorn beside Noganex at equal size: prefill and decode throughput and per-kernel rooflines (one GPU)")
     args = ap.parse_args()
     if args.warmup < 3:
         args.warmup = 3
@@ -1413,6 +1433,8 @@ def main():
         return run_noganex_compare(args)
     if args.nasozen_compare:
         return run_nasozen_compare(args)
+    if args.nomalorn_compare:
+        return run_nomalorn_compare(args)
     workload = args.workload or DEFAULT_WORKLOAD
     if workload in MIXED_WORKLOADS:
         if args.impl == "reference":

@@ -99,8 +99,21 @@ def nasozen_config(name: str) -> dict:
     return {"architecture": "Nasozen", "layers": layers, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "streams": 3, "vocab": 32000, "width": W}
 
 
+def nomalorn_config(name: str) -> dict:
+    """Three layer runs (two layers, the second one twice) at the widths of the `noganex-w*` partners: attention (chunks of 2048, half
+    of each head rotated, a gate per head) beside the delta rule with a decay per key channel (four taps), and a squared-ReLU MLP of
+    four times the width: raw config.json of the Nomalorn family."""
+    W = {"nomalorn-w2048": 2048, "nomalorn-w4096": 4096}[name]
+    left = {"dim": 128, "heads": W // 128, "kv_heads": W // 512, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 2048},
+            "rot": {"base": 1000000.0, "dims": 64}}
+    right = {"conv": 4, "dim": 128, "heads": W // 128, "kv_heads": W // 256, "vdim": 128}
+    layer = {"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": {"kind": "dense", "ff": W * 4}}
+    return {"architecture": "Nomalorn", "layers": [layer, layer], "loop": {"start": 1, "stop": 2, "times": 2}, "norm": {"eps": 1e-5},
+            "vocab": 32000, "width": W}
+
+
 class SyntheticHybridWeights:
-    """Seeded random tensors of a Fetotar, Dubesun, Noganex or Nasozen configuration, generated on the device by name (the `get_tensor`
+    """Seeded random tensors of a Fetotar, Dubesun, Noganex, Nasozen or Nomalorn configuration, generated on the device by name (the `get_tensor`
     side of `Weights`)."""
 
     def __init__(self, raw_config: dict, device, dtype, process_group, seed: int = 1234):
@@ -110,6 +123,8 @@ class SyntheticHybridWeights:
             from ..models.custom_modeling.noganex_modeling import tensor_shapes
         elif raw_config.get("architecture") == "Nasozen":
             from ..models.custom_modeling.nasozen_modeling import tensor_shapes
+        elif raw_config.get("architecture") == "Nomalorn":
+            from ..models.custom_modeling.nomalorn_modeling import tensor_shapes
         else:
             from ..models.custom_modeling.fetotar_modeling import tensor_shapes
         self.shapes, self.device, self.dtype, self.process_group, self.seed = tensor_shapes(raw_config), device, dtype, process_group, seed
@@ -128,7 +143,7 @@ class SyntheticHybridWeights:
         elif len(shape) == 2:
             std = 0.5 if leaf.endswith("conv") else 1.0 / (shape[1] ** 0.5)
             t = torch.empty(shape, dtype=torch.float32, device=self.device).normal_(0.0, std, generator=gen)
-        elif leaf in ("mix.A_log", "mix.dt_bias"):
+        elif leaf.split(".")[-1] in ("A_log", "dt_bias"):
             t = torch.rand(shape, generator=gen, device=self.device) * 2.0 - 2.0
         elif leaf == "mix.f.b":
             t = torch.full(shape, 3.0, device=self.device)
