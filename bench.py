@@ -1361,7 +1361,7 @@ def run_nomalorn_compare(args):
     results = []
     for width in env["widths"]:
         raw = nomalorn_config(f"nomalorn-w{width}")
-        names = ["linear", "embed_scale", "branches_step", "causal_conv", "qk_rot_prepare", "talk_attn", "heads_turn_gate", "delta_scan",
+        names = ["linear", "embed_scale", "branches_step", "qk_rot_prepare", "talk_attn", "heads_turn_gate", "delta_prepare", "delta_rows_scan",
                  "group_rmsnorm_gate", "ff_act", "rmsnorm_rows"]
         cfg = nomalorn_modeling.NomalornConfig(raw)
         r = _stream_family_measure(raw, cfg, names, PB, PL, DB, DL, K, Wm, timed, lib)
@@ -1380,15 +1380,15 @@ def run_nomalorn_compare(args):
         dense_w, head_w = sum(run_w), shapes["embed"][0] * shapes["embed"][1]
         lin_flops = 2 * T * dense_w + 2 * PB * head_w
         pre, dk = r["pre_ops"], r["dec_k"]
-        a_us, s_us, g_us, b_us = us(dk, "talk_attn"), us(dk, "delta_scan"), dk.get("gemm_f16_kernel", 0.0), us(dk, "branches_step")
+        a_us, s_us, g_us, b_us = us(dk, "talk_attn"), us(dk, "delta_step", "delta_chunk"), dk.get("gemm_f16_kernel", 0.0), us(dk, "branches_step")
         kernels = {
             "talk_attn prefill": {"ms": pre["talk_attn"], "tflops": attn_flops / pre["talk_attn"] / 1e9,
                                   "of_measured_tensor": attn_flops / (pre["talk_attn"] * 1e-3) / tens},
             "talk_attn decode": {"us": a_us, "of_measured_hbm": DB * ctx * attn_row * 2 / (max(a_us, 1e-9) * 1e-6) / hbm},
-            "delta_scan prefill": {"ms": pre["delta_scan"], "tokens_per_s_per_layer": T * len(right) / (pre["delta_scan"] * 1e-3),
-                                   "fp32_tflops": scan_flops / pre["delta_scan"] / 1e9,
-                                   "of_measured_hbm": (T * scan_in + PB * state_b / 2) / (pre["delta_scan"] * 1e-3) / hbm},
-            "delta_scan decode": {"us": s_us, "of_measured_hbm": DB * state_b / (max(s_us, 1e-9) * 1e-6) / hbm},
+            "delta_rows_scan prefill": {"ms": pre["delta_rows_scan"], "tokens_per_s_per_layer": T * len(right) / (pre["delta_rows_scan"] * 1e-3),
+                                   "fp32_tflops": scan_flops / pre["delta_rows_scan"] / 1e9,
+                                   "of_measured_hbm": (T * scan_in + PB * state_b / 2) / (pre["delta_rows_scan"] * 1e-3) / hbm},
+            "delta_rows_scan decode": {"us": s_us, "of_measured_hbm": DB * state_b / (max(s_us, 1e-9) * 1e-6) / hbm},
             "branches_step prefill": {"ms": pre["branches_step"], "of_measured_hbm": T * stream_b / (pre["branches_step"] * 1e-3) / hbm},
             "branches_step decode": {"us": b_us, "launches": 1 + sum(2 if l["mlp"] else 1 for l in runs),
                                      "of_measured_hbm": DB * stream_b / (max(b_us, 1e-9) * 1e-6) / hbm},

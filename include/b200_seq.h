@@ -122,13 +122,28 @@ int b200_seq_cast_rows(const float* x, void* out, int dt, int64_t n, void* strea
 /* rows [g | u] (type dt, 2F wide) -> act(g) * u; act 0: SiLU, 1: GELU in its tanh form */
 int b200_seq_ff_gate(const void* gu, void* out, int dt, int64_t rows, int64_t F, int act, void* stream);
 /* gated delta rule over fp32 state slots S [slots, H, dk, dv]: per token S <- g S, u = beta (v - S^T k), S <- S + k u^T, y = S^T q; q and k
- * (kv_heads x dk, shared by H / kv_heads heads) are made unit vectors, q times q_scale; beta = sigmoid(raw[col_b + h]); decay per head,
+ * (kv_heads x dk, shared by H / kv_heads heads) are made unit vectors, q times q_scale; beta = sigmoid(raw[col_b + h]),
+ * g = exp(-exp(A_log[h]) softplus(raw[col_a + h] + dt_bias[h])); c holds the activated q / k / v columns; y fp32 [T, H * dv] */
+int b200_seq_delta_scan(const float* c, int64_t ldc, int col_q, int col_k, int col_v, const float* raw, int64_t ldr, int col_b, int col_a,
+                        const void* A_log, const void* dt_bias, int dt, float q_scale, float* S_state, const int32_t* state_slots,
+                        const int32_t* cu_q, const int64_t* position_ids, float* y, int64_t ld_y, int B, int H, int kv_heads, int dk, int dv,
+                        void* stream);
+/* gated delta rule in two launches, four tokens at a time, with a decay per head or per head and key channel: per token S <- g S,
+ * u = beta (v - S^T k), S <- S + k u^T, y = S^T q; S fp32 [slots, H, dk, dv].
+ * b200_seq_delta_prepare: u fp32 holds the projected q / k (kv_heads x dk each) and v (H x dv) columns from col0; a depth-wise causal
+ * convolution (w [columns, taps], no bias; conv_state fp32 [slots, max(taps - 1, 1), columns] supplies and receives the inputs of other
+ * steps) and SiLU; q and k become unit vectors, q times q_scale; beta = sigmoid(raw[col_b + h]); decay per head,
  * g = exp(-exp(A_log[h]) softplus(dec[col_a + h] + dt_bias[h])), or (channels != 0) per head and key channel n, acting on row n of S,
- * g = exp(-exp(A_log[h]) softplus(dec[col_a + h dk + n] + dt_bias[h dk + n])); c holds the activated q / k / v columns; y fp32 [T, H * dv] */
-int b200_seq_delta_scan(const float* c, int64_t ldc, int col_q, int col_k, int col_v, const float* raw, int64_t ldr, int col_b, const float* dec,
-                        int64_t ldd, int col_a, int channels, const void* A_log, const void* dt_bias, int dt, float q_scale, float* S_state,
-                        const int32_t* state_slots, const int32_t* cu_q, const int64_t* position_ids, float* y, int64_t ld_y, int B, int H,
-                        int kv_heads, int dk, int dv, void* stream);
+ * g = exp(-exp(A_log[h]) softplus(dec[col_a + h dk + n] + dt_bias[h dk + n])) -> out fp32 [T, b200_seq_delta_row_width].
+ * b200_seq_delta_rows_scan: advances S over the prepared rows -> y fp32 [T, H * dv] (q / k shared by H / kv_heads heads) */
+int b200_seq_delta_row_width(int H, int kv_heads, int dk, int dv, int channels);
+int b200_seq_delta_prepare(const float* u, int64_t ld, int col0, int taps, const void* w, float* conv_state, const int32_t* state_slots,
+                           const int32_t* seq_of_token, const int32_t* cu_q, const int64_t* position_ids, const float* raw, int64_t ldr,
+                           int col_b, const float* dec, int64_t ldd, int col_a, int channels, const void* A_log, const void* dt_bias, int dt,
+                           float q_scale, float* out, int64_t T, int B, int H, int kv_heads, int dk, int dv, void* stream);
+int b200_seq_delta_rows_scan(const float* pre, int channels, float* S_state, const int32_t* state_slots, const int32_t* cu_q,
+                        const int64_t* position_ids, float* y, int64_t ld_y, int64_t T, int B, int H, int kv_heads, int dk, int dv,
+                        void* stream);
 /* per token: RMS norm over the whole q projection (H * d columns) and the whole k projection (G * d) when whole_norm != 0 (weights per
  * column, may be NULL), rotation of the first `rot` columns of every head, column i paired with i + rot / 2 (cos / sin fp32
  * [positions, rot / 2]); keys and values to the token-major cache row [k_off: G * d | v_off: G * dv], queries to q_out fp32 [T, H * d].

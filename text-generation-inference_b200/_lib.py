@@ -158,7 +158,11 @@ SEQ_SIGNATURES = {
     "b200_seq_gated_rms_add": (_I, [_P, _P, _P, _I, _P, _P, _L, _L, _F, _P]),
     "b200_seq_cast_rows": (_I, [_P, _P, _I, _L, _P]),
     "b200_seq_ff_gate": (_I, [_P, _P, _I, _L, _L, _I, _P]),
-    "b200_seq_delta_scan": (_I, [_P, _L, _I, _I, _I, _P, _L, _I, _P, _L, _I, _I, _P, _P, _I, _F, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P]),
+    "b200_seq_delta_scan": (_I, [_P, _L, _I, _I, _I, _P, _L, _I, _I, _P, _P, _I, _F, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P]),
+    "b200_seq_delta_row_width": (_I, [_I, _I, _I, _I, _I]),
+    "b200_seq_delta_prepare": (_I, [_P, _L, _I, _I, _P, _P, _P, _P, _P, _P, _P, _L, _I, _P, _L, _I, _I, _P, _P, _I, _F, _P, _L, _I, _I, _I, _I, _I,
+                                    _P]),
+    "b200_seq_delta_rows_scan": (_I, [_P, _I, _P, _P, _P, _P, _P, _L, _L, _I, _I, _I, _I, _I, _P]),
     "b200_seq_qk_rot_prepare": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _P, _I, _F, _P, _P, _I, _P, _P, _P, _I, _L, _I, _I, _P, _L, _P, _P, _I,
                                      _I, _P]),
     "b200_seq_talk_attn": (_I, [_P, _P, _I, _L, _I, _I, _P, _L, _P, _P, _I, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _P]),

@@ -456,21 +456,53 @@ def ff_gate(gate_up: torch.Tensor, act: int) -> torch.Tensor:
 
 
 def delta_scan(c: torch.Tensor, col_q: int, col_k: int, col_v: int, raw: torch.Tensor, col_b: int, col_a: int, A_log: torch.Tensor,
-               dt_bias: torch.Tensor, q_scale: float, S: torch.Tensor, step: RaggedStep, H: int, kv_heads: int, dk: int, dv: int,
-               dec: Optional[torch.Tensor] = None, channels: bool = False) -> torch.Tensor:
+               dt_bias: torch.Tensor, q_scale: float, S: torch.Tensor, step: RaggedStep, H: int, kv_heads: int, dk: int, dv: int) -> torch.Tensor:
     """Gated delta rule -> y fp32 [T, H * dv]; S fp32 [slots, H, dk, dv] advanced in place.  c fp32: activated q / k (kv_heads x dk
-    each) and v (H x dv) columns; raw fp32: write-strength logits, one per head, at col_b; decay logits in `dec` (default: raw) from
-    col_a, one per head, or with `channels` one per head and key channel (H x dk; dt_bias alike): row n of S decays at rate n."""
-    dec = raw if dec is None else dec
-    _cuda(c, raw, dec, S, A_log, dt_bias)
-    assert c.dtype == torch.float32 and raw.dtype == torch.float32 and dec.dtype == torch.float32 and S.dtype == torch.float32 and S.is_contiguous()
-    assert c.stride(1) == 1 and raw.stride(1) == 1 and dec.stride(1) == 1 and A_log.dtype == dt_bias.dtype
-    assert A_log.numel() == H and dt_bias.numel() == (H * dk if channels else H)
+    each) and v (H x dv) columns; raw fp32: write-strength logits at col_b and decay logits at col_a, one per head."""
+    _cuda(c, raw, S, A_log, dt_bias)
+    assert c.dtype == torch.float32 and raw.dtype == torch.float32 and S.dtype == torch.float32 and S.is_contiguous()
+    assert c.stride(1) == 1 and raw.stride(1) == 1 and A_log.dtype == dt_bias.dtype
     y = torch.empty(step.T, H * dv, dtype=torch.float32, device=c.device)
     _lib.check_seq(_lib.load_seq().b200_seq_delta_scan(
-        _ptr(c), c.stride(0), col_q, col_k, col_v, _ptr(raw), raw.stride(0), col_b, _ptr(dec), dec.stride(0), col_a, int(channels), _ptr(A_log),
-        _ptr(dt_bias), _dt(A_log), float(q_scale), _ptr(S), _ptr(step.state_slots), _ptr(step.cu_q), _ptr(step.position_ids), _ptr(y), y.stride(0),
-        step.B, H, kv_heads, dk, dv, _stream()), "seq_delta_scan")
+        _ptr(c), c.stride(0), col_q, col_k, col_v, _ptr(raw), raw.stride(0), col_b, col_a, _ptr(A_log), _ptr(dt_bias), _dt(A_log), float(q_scale),
+        _ptr(S), _ptr(step.state_slots), _ptr(step.cu_q), _ptr(step.position_ids), _ptr(y), y.stride(0), step.B, H, kv_heads, dk, dv, _stream()),
+        "seq_delta_scan")
+    return y
+
+
+def delta_prepare(u: torch.Tensor, col0: int, conv_w: torch.Tensor, conv_state: torch.Tensor, raw: torch.Tensor, col_b: int, dec: torch.Tensor,
+                  col_a: int, A_log: torch.Tensor, dt_bias: torch.Tensor, q_scale: float, step: RaggedStep, H: int, kv_heads: int, dk: int, dv: int,
+                  channels: bool) -> torch.Tensor:
+    """What the gated delta rule needs of every token and the memory has no part in -> fp32 rows for `delta_rows_scan`.  u fp32: projected q / k
+    (kv_heads x dk each) and v (H x dv) columns from col0; conv_w [columns, taps]: their causal convolution, followed by SiLU, with
+    conv_state fp32 [slots, taps - 1, columns] as in causal_conv; q and k become unit vectors, q times q_scale.  raw fp32:
+    write-strength logits, one per head, at col_b; dec fp32: decay logits from col_a, one per head, or with `channels` one per head
+    and key channel (H x dk; dt_bias alike): row n of the memory decays at rate n."""
+    _cuda(u, conv_w, conv_state, raw, dec, A_log, dt_bias)
+    columns = 2 * kv_heads * dk + H * dv
+    for t in (u, raw, dec):
+        assert t.dtype == torch.float32 and t.stride(1) == 1
+    assert conv_w.shape[0] == columns and conv_w.is_contiguous() and conv_state.dtype == torch.float32 and conv_state.is_contiguous()
+    assert conv_state.shape[1:] == (max(conv_w.shape[1] - 1, 1), columns)
+    assert A_log.dtype == dt_bias.dtype == conv_w.dtype and A_log.numel() == H and dt_bias.numel() == (H * dk if channels else H)
+    lib = _lib.load_seq()
+    out = torch.empty(step.T, lib.b200_seq_delta_row_width(H, kv_heads, dk, dv, int(channels)), dtype=torch.float32, device=u.device)
+    _lib.check_seq(lib.b200_seq_delta_prepare(
+        _ptr(u), u.stride(0), col0, conv_w.shape[1], _ptr(conv_w), _ptr(conv_state), _ptr(step.state_slots), _ptr(step.seq_of_token), _ptr(step.cu_q),
+        _ptr(step.position_ids), _ptr(raw), raw.stride(0), col_b, _ptr(dec), dec.stride(0), col_a, int(channels), _ptr(A_log), _ptr(dt_bias),
+        _dt(A_log), float(q_scale), _ptr(out), step.T, step.B, H, kv_heads, dk, dv, _stream()), "seq_delta_prepare")
+    return out
+
+
+def delta_rows_scan(rows: torch.Tensor, S: torch.Tensor, step: RaggedStep, H: int, kv_heads: int, dk: int, dv: int, channels: bool) -> torch.Tensor:
+    """Gated delta rule over rows as `delta_prepare` leaves them -> y fp32 [T, H * dv]; S fp32 [slots, H, dk, dv] advanced in place: per token
+    S <- g S, u = beta (v - S^T k), S <- S + k u^T, y = S^T q."""
+    _cuda(rows, S)
+    assert rows.dtype == torch.float32 and rows.is_contiguous() and S.dtype == torch.float32 and S.is_contiguous() and S.shape[1:] == (H, dk, dv)
+    y = torch.empty(step.T, H * dv, dtype=torch.float32, device=rows.device)
+    _lib.check_seq(_lib.load_seq().b200_seq_delta_rows_scan(_ptr(rows), int(channels), _ptr(S), _ptr(step.state_slots), _ptr(step.cu_q),
+                                                       _ptr(step.position_ids), _ptr(y), y.stride(0), step.T, step.B, H, kv_heads, dk, dv,
+                                                       _stream()), "seq_delta_rows_scan")
     return y
 
 

@@ -648,9 +648,9 @@ class ChannelDeltaMixer(nn.Module):
             raise NotImplementedError("ChannelDeltaMixer: the result is not scaled before its output projection")
         C, R = self.channels, self.rank
         low = ops.linear(ops.ff_act(u[:, col0 + C:col0 + C + R], ops.ACT_NONE, out_dtype=self.dtype), self.w_low, out_dtype=torch.float32)
-        c = ops.causal_conv(u, col0, C, self.conv_w, None, state["conv"], step, act_silu=True)
-        y = ops.delta_scan(c, 0, self.cqk, 2 * self.cqk, u, col0 + C + R, 0, self.A_log, self.dt_bias, self.d ** -0.5, state["S"], step,
-                           self.H, self.G, self.d, self.dv, dec=low, channels=True)
+        rows = ops.delta_prepare(u, col0, self.conv_w, state["conv"], u, col0 + C + R, low, 0, self.A_log, self.dt_bias, self.d ** -0.5, step,
+                                 self.H, self.G, self.d, self.dv, channels=True)
+        y = ops.delta_rows_scan(rows, state["S"], step, self.H, self.G, self.d, self.dv, channels=True)
         ops.group_rmsnorm_gate(y, self.norm_w, self.H, self.eps, self.dtype, gate=low[:, self.n:], gate_kind=ops.GATE_SIGMOID_AFTER, out=out)
 
     def forward(self, h: torch.Tensor, step: ops.RaggedStep, pages, state: Dict[str, torch.Tensor], max_s: int) -> torch.Tensor:
