@@ -131,7 +131,7 @@ int b200_seq_delta_scan(const float* c, int64_t ldc, int col_q, int col_k, int c
 /* gated delta rule in two launches, four tokens at a time, with a decay per head or per head and key channel: per token S <- g S,
  * u = beta (v - S^T k), S <- S + k u^T, y = S^T q; S fp32 [slots, H, dk, dv].
  * b200_seq_delta_prepare: u fp32 holds the projected q / k (kv_heads x dk each) and v (H x dv) columns from col0; a depth-wise causal
- * convolution (w [columns, taps], no bias; conv_state fp32 [slots, max(taps - 1, 1), columns] supplies and receives the inputs of other
+ * convolution (w [taps, columns], no bias; conv_state fp32 [slots, max(taps - 1, 1), columns] supplies and receives the inputs of other
  * steps) and SiLU; q and k become unit vectors, q times q_scale; beta = sigmoid(raw[col_b + h]); decay per head,
  * g = exp(-exp(A_log[h]) softplus(dec[col_a + h] + dt_bias[h])), or (channels != 0) per head and key channel n, acting on row n of S,
  * g = exp(-exp(A_log[h]) softplus(dec[col_a + h dk + n] + dt_bias[h dk + n])) -> out fp32 [T, b200_seq_delta_row_width].

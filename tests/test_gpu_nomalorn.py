@@ -129,7 +129,7 @@ def test_delta_memory_alone(H, G, d, dv, channels):
                 st = _step([(at[i], n) for i, n in entries], [[0] * 3 for _ in entries], slots=[slot[i] for i, _ in entries])
                 parts = [[t[at[i]:at[i] + n] for t in seqs[i]] for i, n in entries]
                 u, raw, dec = (torch.cat([p[j] for p in parts]).to(DEV) for j in range(3))
-                rows = ops.delta_prepare(u, 0, conv_w.to(DEV), cs, raw, 3, dec, 2, A_log.to(DEV), dt_bias.to(DEV), d ** -0.5, st, H, G, d, dv, channels)
+                rows = ops.delta_prepare(u, 0, conv_w.t().contiguous().to(DEV), cs, raw, 3, dec, 2, A_log.to(DEV), dt_bias.to(DEV), d ** -0.5, st, H, G, d, dv, channels)
                 y = ops.delta_rows_scan(rows, S, st, H, G, d, dv, channels)
                 o = 0
                 for i, n in entries:
@@ -169,7 +169,7 @@ def test_delta_convolution_inputs_across_steps(taps):
         at, got = 0, []
         for n in cuts:
             st = _step([(at, n)], [[0] * 2], slots=[1])
-            got.append(ops.delta_prepare(u[at:at + n].to(DEV), 0, conv_w.to(DEV), cs, raw[at:at + n].to(DEV), 3, dec[at:at + n].to(DEV), 2, A_log.to(DEV),
+            got.append(ops.delta_prepare(u[at:at + n].to(DEV), 0, conv_w.t().contiguous().to(DEV), cs, raw[at:at + n].to(DEV), 3, dec[at:at + n].to(DEV), 2, A_log.to(DEV),
                                          dt.to(DEV), d ** -0.5, st, H, G, d, dv, True).cpu().double())
             at += n
         got = torch.cat(got)[:, :want.shape[1]]

@@ -25,7 +25,7 @@
 namespace b200 {
 namespace seq {
 
-constexpr int kDeltaMaxTaps = 8, kPrepThreads = 256, kPrepSpan = 128;  // channels per warp task
+constexpr int kDeltaMaxTaps = 8, kPrepThreads = 256, kPrepSpan = 128, kPrepParts = 2;  // channels per warp task; blocks per token of a long step
 
 // columns of a prepared row
 struct DeltaRow {
@@ -41,29 +41,36 @@ __host__ __device__ inline DeltaRow delta_row(int H, int G, int dk, int dv, bool
   return r;
 }
 
-// SiLU of the causal convolution of channel c at position p; a token alone in its step (`shift`) moves the state on by one input
-template <typename TP>
-__device__ __forceinline__ float conv_silu_at(const float* __restrict__ u, int64_t ld, int col0, int C, int taps, const TP* __restrict__ w, float* st,
-                                              int row0, int64_t s, int64_t p, int c, bool shift) {
-  float acc = 0.f;
-  for (int j = 0; j < taps; ++j) {
-    const int64_t pp = p - (taps - 1) + j;
-    float val = 0.f;
-    if (pp >= s) val = u[(row0 + (pp - s)) * ld + col0 + c];
-    else if (pp >= 0) val = st[(pp - s + taps - 1) * C + c];
-    acc = fmaf(ldf(w + (int64_t)c * taps + j), val, acc);
-    if (shift && j > 0) st[(int64_t)(j - 1) * C + c] = val;   // entry j - 1 was read one iteration ago
+// Where the inputs of one token's convolution lie: a row of this step, an entry of the sequence's state, or nowhere (before position 0).
+// The rows serve every channel, so they are found once per token.
+template <int TAPS>
+struct ConvInputs {
+  const float* src[TAPS];
+};
+
+// SiLU of channel c's convolution (w [taps, C]); a token alone in its step (`shift`) moves the state st [taps - 1, C] on by one input
+template <typename TP, int TAPS>
+__device__ __forceinline__ float conv_silu_at(const ConvInputs<TAPS>& in, const TP* __restrict__ w, float* st, int C, int taps, int c, bool shift) {
+  float val[TAPS], acc = 0.f;
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) val[j] = (j < taps && in.src[j]) ? in.src[j][c] : 0.f;
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j)
+    if (j < taps) acc = fmaf(ldf(w + j * C + c), val[j], acc);
+  if (shift) {
+#pragma unroll
+    for (int j = 1; j < TAPS; ++j)
+      if (j < taps) st[(j - 1) * C + c] = val[j];
   }
   return silu_f(acc);
 }
 
-template <typename TP>
-__global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(
-    const float* __restrict__ u, int64_t ld, int col0, int taps, const TP* __restrict__ w, float* conv_state, int shift,
-    const int32_t* __restrict__ state_slots, const int32_t* __restrict__ seq_of_token, const int32_t* __restrict__ cu_q,
-    const int64_t* __restrict__ position_ids, const float* __restrict__ raw, int64_t ldr, int col_b, const float* __restrict__ dec, int64_t ldd,
-    int col_a, int channels, const TP* __restrict__ A_log, const TP* __restrict__ dt_bias, float q_scale, float* __restrict__ out, int H, int G,
-    int dk, int dv) {
+template <typename TP, int TAPS>  // taps <= TAPS
+__global__ void __launch_bounds__(kPrepThreads, TAPS <= 4 ? 4 : 2) delta_prepare_kernel(
+    const float* u, int64_t ld, int col0, int taps, const TP* __restrict__ w, float* conv_state, int shift, const int32_t* __restrict__ state_slots,
+    const int32_t* __restrict__ seq_of_token, const int32_t* __restrict__ cu_q, const int64_t* __restrict__ position_ids, const float* __restrict__ raw,
+    int64_t ldr, int col_b, const float* __restrict__ dec, int64_t ldd, int col_a, int channels, const TP* __restrict__ A_log,
+    const TP* __restrict__ dt_bias, float q_scale, float* __restrict__ out, int H, int G, int dk, int dv) {
   pdl_launch_dependents();
   pdl_wait();
   const int64_t t = blockIdx.x;
@@ -72,6 +79,12 @@ __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(
   const int64_t s = position_ids[row0], p = position_ids[t];
   const int C = 2 * G * dk + H * dv;
   float* st = conv_state + (int64_t)state_slots[b] * (taps > 1 ? taps - 1 : 1) * C;
+  ConvInputs<TAPS> in;
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) {
+    const int64_t pp = p - (taps - 1) + j;
+    in.src[j] = pp >= s ? u + (row0 + (pp - s)) * ld + col0 : (pp >= 0 ? st + (pp - s + taps - 1) * C : nullptr);
+  }
   const DeltaRow lay = delta_row(H, G, dk, dv, channels != 0);
   float* row = out + t * lay.width;
   const int n_vec = 2 * G, n_v = (H * dv + kPrepSpan - 1) / kPrepSpan, n_dec = channels ? H * dk : H, n_g = (n_dec + kPrepSpan - 1) / kPrepSpan;
@@ -82,7 +95,7 @@ __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
         const int n = lane + 32 * i;
-        x[i] = n < dk ? conv_silu_at(u, ld, col0, C, taps, w, st, row0, s, p, task * dk + n, shift != 0) : 0.f;
+        x[i] = n < dk ? conv_silu_at<TP, TAPS>(in, w, st, C, taps, task * dk + n, shift != 0) : 0.f;
         sum = fmaf(x[i], x[i], sum);
       }
       const float r = (task < G ? q_scale : 1.f) / sqrtf(warp_sum(sum) + 1e-6f);
@@ -92,13 +105,25 @@ __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(
         if (n < dk) row[task * dk + n] = x[i] * r;
       }
     } else if (task < n_vec + n_v) {
-      const int c1 = min(H * dv, (task - n_vec + 1) * kPrepSpan);
-      for (int c = (task - n_vec) * kPrepSpan + lane; c < c1; c += 32)
-        row[lay.v + c] = conv_silu_at(u, ld, col0, C, taps, w, st, row0, s, p, 2 * G * dk + c, shift != 0);
+      const int first = (task - n_vec) * kPrepSpan + lane;
+#pragma unroll
+      for (int i = 0; i < kPrepSpan / 32; ++i) {
+        const int c = first + 32 * i;
+        if (c < H * dv) row[lay.v + c] = conv_silu_at<TP, TAPS>(in, w, st, C, taps, 2 * G * dk + c, shift != 0);
+      }
     } else if (task < n_vec + n_v + n_g) {
-      const int first = (task - n_vec - n_v) * kPrepSpan, c1 = min(n_dec, first + kPrepSpan);
-      for (int c = first + lane; c < c1; c += 32)
-        row[lay.g + c] = expf(-expf(ldf(A_log + (channels ? c / dk : c))) * softplus_f(dec[t * ldd + col_a + c] + ldf(dt_bias + c)));
+      const int first = (task - n_vec - n_v) * kPrepSpan + lane;
+      float z[kPrepSpan / 32];
+#pragma unroll
+      for (int i = 0; i < kPrepSpan / 32; ++i) {
+        const int c = first + 32 * i;
+        z[i] = c < n_dec ? dec[t * ldd + col_a + c] + ldf(dt_bias + c) : 0.f;
+      }
+#pragma unroll
+      for (int i = 0; i < kPrepSpan / 32; ++i) {
+        const int c = first + 32 * i;
+        if (c < n_dec) row[lay.g + c] = expf(-expf(ldf(A_log + (channels ? c / dk : c))) * softplus_f(z[i]));
+      }
     } else {
       const int first = (task - n_vec - n_v - n_g) * kPrepSpan, c1 = min(H, first + kPrepSpan);
       for (int h = first + lane; h < c1; h += 32) row[lay.b + h] = sigmoid_f(raw[t * ldr + col_b + h]);
@@ -147,6 +172,22 @@ __device__ __forceinline__ void halve(float* v, int off, bool upper) {
     const float send = upper ? v[i] : v[i + N / 2], keep = upper ? v[i + N / 2] : v[i];
     v[i] = keep + __shfl_xor_sync(0xffffffffu, send, off);
   }
+}
+
+// the same where every lane has put the values it keeps first
+template <int N>
+__device__ __forceinline__ void fold(float* v, int off) {
+#pragma unroll
+  for (int i = 0; i < N / 2; ++i) v[i] += __shfl_xor_sync(0xffffffffu, v[i + N / 2], off);
+}
+
+// o[x] = f[x ^ (lo + 2 hi)]; its own inverse
+__device__ __forceinline__ void permute4(float4 f, bool lo, bool hi, float* o) {
+  const float a = lo ? f.y : f.x, b = lo ? f.x : f.y, c = lo ? f.w : f.z, d = lo ? f.z : f.w;
+  o[0] = hi ? c : a;
+  o[1] = hi ? d : b;
+  o[2] = hi ? a : c;
+  o[3] = hi ? b : d;
 }
 
 template <int NR>  // state rows per lane: dk <= 16 NR
@@ -215,10 +256,11 @@ __global__ void __launch_bounds__(256, NR <= 8 ? 2 : 1) delta_chunk_kernel(
     cp_async_commit();
   };
 
-  // this thread's part of the memory: rows rl + 16 i, columns c0 .. c0 + 3 of the block's
+  // this thread's part of the memory: rows rl + 16 i, columns c0 .. c0 + 3 of the block's.  Entry x of S[i] is column c0 + (x ^ perm): with
+  // a lane's own column order a reduction over lanes always keeps the lower half of what it has and sends the upper half
   const int rl = lane & 15, c0 = w * kColsPerWarp + (lane >> 4) * 4;
   const bool b3 = lane & 8, b2 = lane & 4, b1 = lane & 2, b0 = lane & 1;
-  const int my_c = c0 + (b3 ? 2 : 0) + (b2 ? 1 : 0);     // the column whose reductions this lane ends up with
+  const int perm = (lane >> 2) & 3, my_c = c0 + perm;    // my_c: the column whose reductions this lane ends up with
   float* Sp = S_state + ((int64_t)state_slots[b] * H + h) * dk * dv + v0;
   load_tile(t_begin, 0);
   float S[NR][4];
@@ -230,12 +272,12 @@ __global__ void __launch_bounds__(256, NR <= 8 ? 2 : 1) delta_chunk_kernel(
       if (vec) {
         if (c0 < live_cols) {
           const float4 f = *reinterpret_cast<const float4*>(Sp + (int64_t)n * dv + c0);
-          S[i][0] = f.x; S[i][1] = f.y; S[i][2] = f.z; S[i][3] = f.w;
+          permute4(f, b2, b3, S[i]);
         }
       } else {
 #pragma unroll
-        for (int c = 0; c < 4; ++c)
-          if (c0 + c < live_cols) S[i][c] = Sp[(int64_t)n * dv + c0 + c];
+        for (int x = 0; x < 4; ++x)
+          if (c0 + (x ^ perm) < live_cols) S[i][x] = Sp[(int64_t)n * dv + c0 + (x ^ perm)];
       }
     }
   }
@@ -317,8 +359,8 @@ __global__ void __launch_bounds__(256, NR <= 8 ? 2 : 1) delta_chunk_kernel(
         }
       }
       // predictions: every group of four lanes ends with the four tokens of one column
-      halve<16>(P, 8, b3);
-      halve<8>(P, 4, b2);
+      fold<16>(P, 8);
+      fold<8>(P, 4);
 #pragma unroll
       for (int j = 0; j < 4; ++j) P[j] += __shfl_xor_sync(0xffffffffu, P[j], 2);
 #pragma unroll
@@ -340,13 +382,10 @@ __global__ void __launch_bounds__(256, NR <= 8 ? 2 : 1) delta_chunk_kernel(
       float U[4][4];   // [token][column]
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        const float x = __shfl_xor_sync(0xffffffffu, um[j], 4);
-        const float lo = b2 ? x : um[j], hi = b2 ? um[j] : x;
-        const float xl = __shfl_xor_sync(0xffffffffu, lo, 8), xh = __shfl_xor_sync(0xffffffffu, hi, 8);
-        U[j][0] = b3 ? xl : lo;
-        U[j][1] = b3 ? xh : hi;
-        U[j][2] = b3 ? lo : xl;
-        U[j][3] = b3 ? hi : xh;
+        U[j][0] = um[j];
+        U[j][1] = __shfl_xor_sync(0xffffffffu, um[j], 4);
+        U[j][2] = __shfl_xor_sync(0xffffffffu, U[j][0], 8);
+        U[j][3] = __shfl_xor_sync(0xffffffffu, U[j][1], 8);
       }
 #pragma unroll
       for (int i = 0; i < NR; ++i) {
@@ -357,8 +396,8 @@ __global__ void __launch_bounds__(256, NR <= 8 ? 2 : 1) delta_chunk_kernel(
           S[i][c] = fmaf(kd.w, U[3][c], fmaf(kd.z, U[2][c], fmaf(kd.y, U[1][c], fmaf(kd.x, U[0][c], ga * S[i][c]))));
       }
       // read-outs: every lane ends with one (token, column)
-      halve<16>(O, 8, b3);
-      halve<8>(O, 4, b2);
+      fold<16>(O, 8);
+      fold<8>(O, 4);
       halve<4>(O, 2, b1);
       halve<2>(O, 1, b0);
       const int j = lane & 3, t = t0 + qd * kQuad + j;
@@ -372,11 +411,13 @@ __global__ void __launch_bounds__(256, NR <= 8 ? 2 : 1) delta_chunk_kernel(
     const int n = rl + kRowLanes * i;
     if (n < dk) {
       if (vec) {
-        if (c0 < live_cols) *reinterpret_cast<float4*>(Sp + (int64_t)n * dv + c0) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
+        float o[4];
+        permute4(make_float4(S[i][0], S[i][1], S[i][2], S[i][3]), b2, b3, o);
+        if (c0 < live_cols) *reinterpret_cast<float4*>(Sp + (int64_t)n * dv + c0) = make_float4(o[0], o[1], o[2], o[3]);
       } else {
 #pragma unroll
-        for (int c = 0; c < 4; ++c)
-          if (c0 + c < live_cols) Sp[(int64_t)n * dv + c0 + c] = S[i][c];
+        for (int x = 0; x < 4; ++x)
+          if (c0 + (x ^ perm) < live_cols) Sp[(int64_t)n * dv + c0 + (x ^ perm)] = S[i][x];
       }
     }
   }
@@ -506,7 +547,7 @@ using namespace b200::seq;
 // floats per prepared row
 extern "C" int b200_seq_delta_row_width(int H, int kv_heads, int dk, int dv, int channels) { return delta_row(H, kv_heads, dk, dv, channels != 0).width; }
 
-// u fp32 [T, ld]: projected q / k (kv_heads x dk each) and v (H x dv) columns from col0; w [2 kv_heads dk + H dv, taps] their convolution;
+// u fp32 [T, ld]: projected q / k (kv_heads x dk each) and v (H x dv) columns from col0; w [taps, 2 kv_heads dk + H dv] their convolution;
 // conv_state fp32 [slots, max(taps - 1, 1), channels of u] advanced in place; raw fp32: write-strength logits, one per head, at col_b; dec
 // fp32: decay logits from col_a, one per head or (channels != 0) dk per head; A_log [H], dt_bias ([H] or [H * dk]), w of element type dt
 // -> out fp32 [T, b200_seq_delta_row_width]
@@ -524,10 +565,15 @@ extern "C" int b200_seq_delta_prepare(const float* u, int64_t ld, int col0, int 
   const int tasks = 2 * kv_heads + (H * dv + kPrepSpan - 1) / kPrepSpan + ((channels ? H * dk : H) + kPrepSpan - 1) / kPrepSpan +
                     (H + kPrepSpan - 1) / kPrepSpan;
   int parts = (tasks + kPrepThreads / 32 - 1) / (kPrepThreads / 32);   // few rows: a warp per task; many: blocks that loop
-  if (T > 1024 && parts > 2) parts = 2;
-  B200_SEQ_DISPATCH(dt, E, B200_LAUNCH((delta_prepare_kernel<E>), dim3((unsigned)T, (unsigned)parts), dim3(kPrepThreads), 0, st, u, ld, col0, taps,
-                                       (const E*)w, conv_state, shift, state_slots, seq_of_token, cu_q, position_ids, raw, ldr, col_b, dec, ldd, col_a,
-                                       channels, (const E*)A_log, (const E*)dt_bias, q_scale, out, H, kv_heads, dk, dv));
+  if (T > 1024 && parts > kPrepParts) parts = kPrepParts;
+#define DPR(N)                                                                                                                                      \
+  B200_SEQ_DISPATCH(dt, E, B200_LAUNCH((delta_prepare_kernel<E, N>), dim3((unsigned)T, (unsigned)parts), dim3(kPrepThreads), 0, st, u, ld, col0, taps, \
+                                       (const E*)w, conv_state, shift, state_slots, seq_of_token, cu_q, position_ids, raw, ldr, col_b, dec, ldd, col_a, \
+                                       channels, (const E*)A_log, (const E*)dt_bias, q_scale, out, H, kv_heads, dk, dv))
+  if (taps <= 2) DPR(2);
+  else if (taps <= 4) DPR(4);
+  else DPR(8);
+#undef DPR
   if (!shift && taps > 1)
     B200_LAUNCH(delta_conv_state_kernel, dim3((unsigned)B, (unsigned)((C + 255) / 256)), dim3(256), 0, st, u, ld, col0, C, taps, conv_state, state_slots,
                 cu_q, position_ids);

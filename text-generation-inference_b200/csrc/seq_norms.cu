@@ -435,6 +435,99 @@ __global__ void ff_act_kernel(const TI* __restrict__ in, int64_t ld_in, TO* __re
   }
 }
 
+// eight consecutive elements as 16-byte accesses
+template <typename T>
+__device__ __forceinline__ void ld8(const T* p, float (&v)[8]) {
+  if constexpr (sizeof(T) == 4) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+  } else {
+    const uint4 a = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[i]));
+      v[2 * i] = f.x;
+      v[2 * i + 1] = f.y;
+    }
+  }
+}
+template <typename T>
+__device__ __forceinline__ void st8(T* p, const float (&v)[8]) {
+  if constexpr (sizeof(T) == 4) {
+    reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+    reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+  } else {
+    uint32_t w[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const __nv_bfloat162 b = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+      w[i] = *reinterpret_cast<const uint32_t*>(&b);
+    }
+    *reinterpret_cast<uint4*>(p) = make_uint4(w[0], w[1], w[2], w[3]);
+  }
+}
+
+// ff_act_kernel for rows of whole 8-element pieces on 16-byte boundaries
+template <typename TI, typename TO, int ACT>
+__global__ void __launch_bounds__(kRowThreads) ff_act_vec_kernel(const TI* __restrict__ in, int64_t ld_in, TO* __restrict__ out, int64_t rows, int F) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const uint32_t per_row = (uint32_t)F / 8;
+  for (int64_t r = blockIdx.x; r < rows; r += gridDim.x)
+    for (uint32_t c = blockIdx.y * kRowThreads + threadIdx.x; c < per_row; c += gridDim.y * kRowThreads) {
+      float v[8];
+      ld8(in + r * ld_in + c * 8, v);
+#pragma unroll
+      for (int k = 0; k < 8; ++k) v[k] = plain_act_f<ACT>(v[k]);
+      st8(out + r * F + c * 8, v);
+    }
+}
+
+// group_rmsnorm_gate_kernel for groups of n <= 512 columns: one warp per (row, group), VEC columns per access, the group held in
+// registers between its statistic and its way out
+template <typename TP, typename TO, int VEC, int PIECES>
+__global__ void __launch_bounds__(kRowThreads) group_rmsnorm_warp_kernel(const float* __restrict__ x, int64_t ldx, const float* __restrict__ gate,
+                                                                         int64_t ldg, int gate_kind, const TP* __restrict__ w, int groups, int n,
+                                                                         float eps, TO* __restrict__ out, int64_t ldo, int64_t items) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t item = (int64_t)blockIdx.x * (kRowThreads / 32) + warp_id();
+  if (item >= items) return;
+  const int64_t t = item / groups;
+  const int c0 = (int)(item % groups) * n;
+  float v[PIECES][VEC], g[PIECES][VEC], q = 0.f;
+#pragma unroll
+  for (int i = 0; i < PIECES; ++i) {
+    const int c = (lane_id() + 32 * i) * VEC;
+    if (c < n) {
+      ld_vec<VEC>(x + t * ldx + c0 + c, v[i]);
+      if (gate_kind) ld_vec<VEC>(gate + t * ldg + c0 + c, g[i]);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) {
+        if (gate_kind == 1) v[i][k] *= silu_f(g[i][k]);
+        q += v[i][k] * v[i][k];
+      }
+    }
+  }
+  const float rstd = 1.f / sqrtf(warp_sum(q) / n + eps);
+#pragma unroll
+  for (int i = 0; i < PIECES; ++i) {
+    const int c = (lane_id() + 32 * i) * VEC;
+    if (c < n) {
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) {
+        float o = v[i][k] * rstd;
+        if (w) o *= ldf(w + c0 + c + k);
+        if (gate_kind == 2) o *= sigmoid_f(g[i][k]);
+        else if (gate_kind == 3) o *= silu_f(g[i][k]);
+        v[i][k] = o;
+      }
+      st_vec<TO, VEC>(out + t * ldo + c0 + c, v[i]);
+    }
+  }
+}
+
 // Attention heads on their way to the output projection: a [T, H, dv] fp32; every head's first `rot` columns are turned by
 // -position (pairs: column i with column i + rot / 2 when `interleaved` is 0, columns 2i and 2i + 1 otherwise; cos / sin
 // [positions, rot / 2]), then the head is multiplied by sigmoid(gate[t, h]) (gate NULL: by 1) and by out_scale -> out rows of
@@ -531,6 +624,29 @@ extern "C" int b200_seq_group_rmsnorm_gate(const float* x, int64_t ldx, const fl
   const int C = groups > 0 ? groups * n : n;
   const int part = groups > 0 ? n : 2048;
   const dim3 grid((unsigned)T, (unsigned)((C + part - 1) / part));
+  // 16-byte accesses when every group starts on a 16-byte boundary (the gate and the typed rows included)
+  const bool vec = groups > 0 && n % 4 == 0 && ldx % 4 == 0 && (gate == nullptr || ldg % 4 == 0) && ldo % 4 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+  if (vec && n <= 512) {
+    const int64_t items = T * groups;
+#define GW_LAUNCH(TP, TO, P)                                                                                                            \
+  B200_LAUNCH((group_rmsnorm_warp_kernel<TP, TO, 4, P>), dim3((unsigned)((items + 7) / 8)), dim3(kRowThreads), 0, st, x, ldx, gate, ldg, gate_kind, \
+              (const TP*)w, groups, n, eps, (TO*)out, ldo, items)
+#define GW(TP, TO)                            \
+  do {                                        \
+    if (n <= 128) GW_LAUNCH(TP, TO, 1);       \
+    else if (n <= 256) GW_LAUNCH(TP, TO, 2);  \
+    else GW_LAUNCH(TP, TO, 4);                \
+  } while (0)
+    if (w_dt == B200_DT_F32 && out_dt == B200_DT_F32) GW(float, float);
+    else if (w_dt == B200_DT_BF16 && out_dt == B200_DT_BF16) GW(__nv_bfloat16, __nv_bfloat16);
+    else if (w_dt == B200_DT_BF16 && out_dt == B200_DT_F32) GW(__nv_bfloat16, float);
+    else { b200_set_last_error("seq_group_rmsnorm_gate: unsupported element types"); return B200_ERR_UNSUPPORTED; }
+#undef GW
+#undef GW_LAUNCH
+    b200_count_launches(1);
+    return B200_OK;
+  }
 #define GN_LAUNCH(TP, TO)                                                                                                                   \
   B200_LAUNCH((group_rmsnorm_gate_kernel<TP, TO>), grid, dim3(kRowThreads), 0, st, x, ldx, gate, ldg, gate_kind, (const TP*)w, groups, part, \
               C, eps, (TO*)out, ldo)
@@ -676,7 +792,16 @@ extern "C" int b200_seq_ff_act(const void* in, int in_dt, int64_t ld_in, void* o
   int64_t blocks = (rows * F + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   if (act < 0 || act > 4) { b200_set_last_error("seq_ff_act: unknown activation"); return B200_ERR_ARG; }
-#define FA(TI, TO, A) B200_LAUNCH((ff_act_kernel<TI, TO, A>), dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, (const TI*)in, ld_in, (TO*)out, rows, (int)F)
+  const size_t in_sz = in_dt == B200_DT_F32 ? 4 : 2;
+  const bool vec = F % 8 == 0 && (ld_in * in_sz) % 16 == 0 && ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+  const int64_t per_row = (F / 8 + kRowThreads - 1) / kRowThreads, many = 148 * 64;
+  const dim3 vgrid((unsigned)(rows < many ? rows : many), (unsigned)(per_row < 8 ? per_row : 8));
+#define FA(TI, TO, A)                                                                                                                              \
+  do {                                                                                                                                             \
+    if (vec) B200_LAUNCH((ff_act_vec_kernel<TI, TO, A>), vgrid, dim3(kRowThreads), 0, (cudaStream_t)stream, (const TI*)in, ld_in, (TO*)out, rows, (int)F); \
+    else FA_PLAIN(TI, TO, A);                                                                                                                      \
+  } while (0)
+#define FA_PLAIN(TI, TO, A) B200_LAUNCH((ff_act_kernel<TI, TO, A>), dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, (const TI*)in, ld_in, (TO*)out, rows, (int)F)
 #define FA_ACT(TI, TO)            \
   do {                            \
     if (act == 0) FA(TI, TO, 0);  \
@@ -691,6 +816,7 @@ extern "C" int b200_seq_ff_act(const void* in, int in_dt, int64_t ld_in, void* o
   else { b200_set_last_error("seq_ff_act: element types must be fp32 -> any or bf16 -> bf16"); return B200_ERR_ARG; }
 #undef FA_ACT
 #undef FA
+#undef FA_PLAIN
   b200_count_launches(1);
   return B200_OK;
 }

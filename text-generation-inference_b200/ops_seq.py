@@ -474,7 +474,7 @@ def delta_prepare(u: torch.Tensor, col0: int, conv_w: torch.Tensor, conv_state: 
                   col_a: int, A_log: torch.Tensor, dt_bias: torch.Tensor, q_scale: float, step: RaggedStep, H: int, kv_heads: int, dk: int, dv: int,
                   channels: bool) -> torch.Tensor:
     """What the gated delta rule needs of every token and the memory has no part in -> fp32 rows for `delta_rows_scan`.  u fp32: projected q / k
-    (kv_heads x dk each) and v (H x dv) columns from col0; conv_w [columns, taps]: their causal convolution, followed by SiLU, with
+    (kv_heads x dk each) and v (H x dv) columns from col0; conv_w [taps, columns]: their causal convolution, followed by SiLU, with
     conv_state fp32 [slots, taps - 1, columns] as in causal_conv; q and k become unit vectors, q times q_scale.  raw fp32:
     write-strength logits, one per head, at col_b; dec fp32: decay logits from col_a, one per head, or with `channels` one per head
     and key channel (H x dk; dt_bias alike): row n of the memory decays at rate n."""
@@ -482,13 +482,13 @@ def delta_prepare(u: torch.Tensor, col0: int, conv_w: torch.Tensor, conv_state: 
     columns = 2 * kv_heads * dk + H * dv
     for t in (u, raw, dec):
         assert t.dtype == torch.float32 and t.stride(1) == 1
-    assert conv_w.shape[0] == columns and conv_w.is_contiguous() and conv_state.dtype == torch.float32 and conv_state.is_contiguous()
-    assert conv_state.shape[1:] == (max(conv_w.shape[1] - 1, 1), columns)
+    assert conv_w.shape[1] == columns and conv_w.is_contiguous() and conv_state.dtype == torch.float32 and conv_state.is_contiguous()
+    assert conv_state.shape[1:] == (max(conv_w.shape[0] - 1, 1), columns)
     assert A_log.dtype == dt_bias.dtype == conv_w.dtype and A_log.numel() == H and dt_bias.numel() == (H * dk if channels else H)
     lib = _lib.load_seq()
     out = torch.empty(step.T, lib.b200_seq_delta_row_width(H, kv_heads, dk, dv, int(channels)), dtype=torch.float32, device=u.device)
     _lib.check_seq(lib.b200_seq_delta_prepare(
-        _ptr(u), u.stride(0), col0, conv_w.shape[1], _ptr(conv_w), _ptr(conv_state), _ptr(step.state_slots), _ptr(step.seq_of_token), _ptr(step.cu_q),
+        _ptr(u), u.stride(0), col0, conv_w.shape[0], _ptr(conv_w), _ptr(conv_state), _ptr(step.state_slots), _ptr(step.seq_of_token), _ptr(step.cu_q),
         _ptr(step.position_ids), _ptr(raw), raw.stride(0), col_b, _ptr(dec), dec.stride(0), col_a, int(channels), _ptr(A_log), _ptr(dt_bias),
         _dt(A_log), float(q_scale), _ptr(out), step.T, step.B, H, kv_heads, dk, dv, _stream()), "seq_delta_prepare")
     return out

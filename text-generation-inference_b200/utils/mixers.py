@@ -619,12 +619,12 @@ class ChannelDeltaMixer(nn.Module):
         pad = a1.new_zeros(self.rank - ra - rg, a1.shape[1])
         self.w_in = torch.cat([get("q"), get("k"), get("v"), a1, g1, pad, get("b")], 0).contiguous()   # -> [q | k | v | latent | beta]
         self.n_in = self.channels + self.rank + self.H
-        self.conv_w = torch.cat([get(f"{n}.conv") for n in ("q", "k", "v")], 0).contiguous()
+        self.conv_w = torch.cat([get(f"{n}.conv") for n in ("q", "k", "v")], 0).t().contiguous()   # [taps, columns]
         self.A_log, self.dt_bias = get("A_log").contiguous(), get("dt_bias").contiguous()
         self.norm_w = get("norm").repeat(self.H).contiguous()                             # one entry per column of the heads
         self.w_o = get("o").contiguous()
         self.dtype = self.w_o.dtype
-        if self.w_in.shape[0] != self.n_in or self.conv_w.shape != (self.channels, self.taps) or a2.shape != (self.n, ra) or \
+        if self.w_in.shape[0] != self.n_in or self.conv_w.shape != (self.taps, self.channels) or a2.shape != (self.n, ra) or \
                 g2.shape != (self.n_out, rg) or self.dt_bias.shape != (self.n,) or self.A_log.shape != (self.H,) or \
                 self.norm_w.shape != (self.n_out,) or self.w_o.shape[1] != self.n_out:
             raise ValueError(f"{prefix}: tensor shapes do not match the head sizes")
