@@ -94,7 +94,7 @@ def _delta_inputs(g, L, H, G, d, dv, channels, wild=False):
 
 
 @pytest.mark.parametrize("H,G,d,dv,channels", [(4, 2, 12, 14, True), (3, 3, 10, 9, True), (2, 1, 72, 80, True), (1, 1, 132, 36, True), (2, 2, 256, 40, True),
-                                               (2, 1, 64, 130, True), (4, 4, 64, 64, True), (6, 2, 16, 200, True), (1, 1, 5, 1, True),
+                                               (2, 1, 64, 130, True), (3, 3, 64, 64, True), (6, 2, 16, 200, True), (1, 1, 5, 1, True),
                                                (4, 2, 12, 14, False), (2, 1, 128, 128, False), (3, 1, 68, 10, False)])
 def test_delta_memory_alone(H, G, d, dv, channels):
     """preparation and memory against the token-by-token recurrence: whole sequences, single rows, ragged groups whose sizes leave one to
@@ -180,7 +180,7 @@ def test_delta_convolution_inputs_across_steps(taps):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("H,G,d,dv,conv,ranks", [(4, 2, 12, 14, 3, (5, 7)), (2, 2, 64, 32, 4, (24, 8)), (3, 1, 20, 70, 1, (60, 13)), (1, 1, 8, 6, 2, (1, 2))])
+@pytest.mark.parametrize("H,G,d,dv,conv,ranks", [(4, 2, 12, 14, 3, (5, 7)), (2, 2, 48, 32, 4, (20, 8)), (3, 1, 20, 70, 1, (60, 13)), (1, 1, 8, 6, 2, (1, 2))])
 def test_channel_delta_mixer_any_cut(H, G, d, dv, conv, ranks, dtype):
     import tgis_b200  # noqa: F401
     from tgis_b200.utils.mixers import ChannelDeltaMixer
@@ -247,7 +247,7 @@ def test_attention_half_any_cut(H, G, d, dv, rot, chunk, dtype):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("H,G,d,dv,chunk", [(6, 3, 10, 14, 100), (8, 1, 16, 80, 64), (8, 2, 32, 48, 33), (16, 4, 16, 96, 150), (2, 2, 64, 112, 17)])
+@pytest.mark.parametrize("H,G,d,dv,chunk", [(6, 3, 10, 14, 100), (6, 2, 16, 80, 70), (8, 2, 32, 48, 33), (16, 4, 16, 96, 150), (2, 2, 64, 112, 17)])
 def test_loud_keys_at_chunk_edges(dtype, H, G, d, dv, chunk):
     """One key is made to win the soft-max of every head: the output must be that key's value when the key is the chunk's first
     position, at a page border or the query itself, and must not move when the key is the last position of the chunk before - for a
