@@ -50,11 +50,12 @@ int b200_seq_latent_prepare(const float* down, int64_t ld_down, int col_c, int c
                             float eps, void* stream);
 /* out[t, h, :R] = sum_j softmax_j((q_abs[t, h] . cache_row(j)) * scale) cache_row(j)[:R], j over (p - window, p] of t's sequence.
  * b200_seq_latent_attn_splits: over how many blocks the tensor-core kernel should split each token's keys for this shape (0: the
- * shape takes the plain kernel) and the fp32 workspace (`partial`) that takes; partial NULL / nsplit <= 1: no split */
+ * shape takes the plain kernel) and the fp32 workspace (`partial`) that takes; partial NULL / nsplit <= 1: no split.  sink fp32 [H]
+ * (NULL: none): exp(sink[h]) joins head h's soft-max denominator (unscaled) and carries no value */
 int b200_seq_latent_attn_splits(int dt, int64_t Tq, int H, int R, int r, int64_t* workspace_floats);
 int b200_seq_latent_attn(const float* q_abs, const void* cache, int dt, const int32_t* block_table, int64_t bt_stride,
                          const int32_t* seq_of_token, const int64_t* position_ids, float* out, int64_t Tq, int H, int R, int r, int window,
-                         float scale, int page, float* partial, int nsplit, void* stream);
+                         float scale, int page, float* partial, int nsplit, const float* sink, void* stream);
 /* SiLU(depth-wise causal convolution) of columns [col0, col0 + C) of u; conv_state [slots, taps - 1, C] read and advanced */
 int b200_seq_causal_conv_silu(const float* u, int64_t ld_u, int col0, int C, int taps, const void* w, const void* bias, int dt,
                               float* conv_state, const int32_t* state_slots, const int32_t* seq_of_token, const int32_t* cu_q,
@@ -102,18 +103,22 @@ int b200_seq_diff_combine(const float* in, void* out, int out_dt, int64_t T, int
  * expert, tiles of 64 rows) that the grouped products and the combine read; plan = b200_seq_moe_plan_ints int32 values */
 int64_t b200_seq_moe_plan_ints(int64_t T, int E, int top);
 int b200_seq_moe_route(const float* logits, int64_t T, int E, int top, int32_t* ids, float* weights, int32_t* plan, void* stream);
-/* C[row] = W[expert(row)] A[gather ? token(row) : row] for the T * top rows of the plan; W [E, N, K] */
+/* C[row] = act(W[expert(row)] A[gather ? token(row) : row]) for the rows of the plan; W [E, N, K]; act 0: none, 1: relu(z)^2 */
 int b200_seq_moe_linear(const void* A, int a_dt, int64_t lda, int gather, const void* W, int w_dt, void* C, int c_dt, int64_t ldc,
-                        int32_t* plan, int64_t T, int E, int top, int64_t N, int64_t K, void* stream);
+                        int32_t* plan, int64_t T, int E, int top, int64_t N, int64_t K, int act, void* stream);
 /* out [T * top, K] = A[token(row)]: compact rows for callers that run one dense product per expert (plan offsets at int E of plan) */
 int b200_seq_moe_gather_rows(const void* A, int dt, int64_t lda, void* out, int32_t* plan, int64_t T, int E, int top, int64_t K, void* stream);
 /* resid += mix + sum_k weights[t, k] y[row(t, k)]; mix and y may be NULL */
 int b200_seq_moe_combine_add(float* resid, const float* mix, const float* y, int64_t ldy, const float* weights, int32_t* plan, int64_t T,
                              int E, int top, int64_t W, void* stream);
 /* mode 0: as b200_seq_moe_route; mode 1: scores = sigmoid(logit), the picks are the largest score + correction[expert] (element type
- * corr_dt, may be NULL), weights = picked score / (sum of the picked scores + 1e-20) * weight_scale */
-int b200_seq_moe_route_scored(const float* logits, int64_t T, int E, int top, int mode, const void* correction, int corr_dt, float weight_scale,
-                              int32_t* ids, float* weights, int32_t* plan, void* stream);
+ * corr_dt, may be NULL), weights = picked score / (sum of the picked scores + 1e-20) * weight_scale; mode 2: the same with
+ * scores = soft-max over all router outputs.  Router outputs E .. E_all - 1 are identity outputs: picked and weighed like experts, but
+ * without a row in the plan; ld: leading dimension of the logits */
+int b200_seq_moe_route_scored(const float* logits, int64_t ld, int64_t T, int E, int E_all, int top, int mode, const void* correction, int corr_dt,
+                              float weight_scale, int32_t* ids, float* weights, int32_t* plan, void* stream);
+/* the plan's row_of [T, top]: compact row of every pick, -1 for an identity output */
+int32_t* b200_seq_moe_row_of(int32_t* plan, int64_t T, int E, int top);
 /* resid (fp32) += v / sqrt(mean v^2 + eps) * w, v = y * sigmoid(gate) (gate NULL: y); typed (type dt, may be NULL) = the updated rows */
 int b200_seq_gated_rms_add(const float* y, const float* gate, const void* w, int dt, float* resid, void* typed, int64_t T, int64_t W, float eps,
                            void* stream);
@@ -148,12 +153,12 @@ int b200_seq_delta_rows_scan(const float* pre, int channels, float* S_state, con
  * column, may be NULL), rotation of the first `rot` columns of every head, column i paired with i + rot / 2 (cos / sin fp32
  * [positions, rot / 2]); keys and values to the token-major cache row [k_off: G * d | v_off: G * dv], queries to q_out fp32 [T, H * d].
  * v_rot > 0: the first v_rot columns of every value head turn by the token's position too (vcos / vsin fp32 [positions, v_rot / 2];
- * pairs are column i with i + v_rot / 2, or columns 2i and 2i + 1 when v_interleaved != 0) */
+ * pairs are column i with i + v_rot / 2, or columns 2i and 2i + 1 when v_interleaved != 0; `interleaved` says the same of q and k) */
 int b200_seq_qk_rot_prepare(const float* src, int64_t ld, int col_q, int col_k, int col_v, int H, int G, int d, int dv, const void* qnorm_w,
                             const void* knorm_w, int whole_norm, float eps, const float* cos_t, const float* sin_t, int rot,
                             const int64_t* position_ids, const int64_t* slot_mapping, void* cache, int dt, int64_t row_width, int k_off,
                             int v_off, float* q_out, int64_t T, const float* vcos_t, const float* vsin_t, int v_rot, int v_interleaved,
-                            void* stream);
+                            int interleaved, void* stream);
 /* attention with the scaled scores mixed over the heads before the soft-max (talk fp32 [H, H], NULL: none); a query at p sees keys
  * j <= p with floor(j / chunk) == floor(p / chunk) (chunk > 0) and p - j < window (window > 0); sink fp32 [H] (NULL: none): exp(sink[h])
  * joins head h's soft-max denominator (after the mix, unscaled) and carries no value; out fp32 [T, H, dv] */
@@ -175,6 +180,14 @@ int b200_seq_streams_step(float* X, int S, const float* init, const float* y, co
 int b200_seq_branches_step(float* x, const float* init, const float* y1, const void* w1, const float* y2, const void* w2, float y_scale,
                            const float* add, const void* step_vec, const void* norm_w, int dt, void* typed, int64_t T, int64_t W, float eps,
                            void* stream);
+/* one fp32 stream whose layers add two halves side by side, x [T, W] in place (or from `init`): x += y1 + sigmoid(gate[t * ld_gate]) * y2
+ * (gate NULL: y2) + sum_k weights[t, k] * (row_of[t, k] >= 0 ? rows[row_of[t, k]] : pass[t]) (top <= 16; pass of type dt), then
+ * typed_a, typed_b (type dt) <- x / sqrt(mean x^2 + eps) * norm_a, * norm_b; every pointer but x may be NULL */
+int b200_seq_halves_step(float* x, const float* init, const float* y1, const float* y2, const float* gate, int64_t ld_gate, const float* rows,
+                         int64_t ld_rows, const float* weights, const int32_t* row_of, int top, const void* pass, const void* norm_a,
+                         const void* norm_b, int dt, void* typed_a, void* typed_b, int64_t T, int64_t W, float eps, void* stream);
+/* z <- cap * tanh(z / cap), n fp32 values in place */
+int b200_seq_soft_cap(float* z, int64_t n, float cap, void* stream);
 /* out (dense rows of type out_dt) = act(in) over rows of F columns with leading dimension ld_in; act 0: SiLU, 1: GELU in its tanh form,
  * 2: tanh, 3: relu(z)^2, 4: none (a copy or a change of type); element types fp32 -> any or bf16 -> bf16 */
 int b200_seq_ff_act(const void* in, int in_dt, int64_t ld_in, void* out, int out_dt, int64_t rows, int64_t F, int act, void* stream);

@@ -138,7 +138,7 @@ SEQ_SIGNATURES = {
     "b200_seq_rms_add": (_I, [_P, _P, _I, _P, _L, _L, _F, _P]),
     "b200_seq_latent_prepare": (_I, [_P, _L, _I, _I, _P, _L, _I, _I, _P, _P, _P, _P, _P, _P, _I, _P, _L, _I, _I, _I, _I, _F, _P]),
     "b200_seq_latent_attn_splits": (_I, [_I, _L, _I, _I, _I, ctypes.POINTER(c_int64)]),
-    "b200_seq_latent_attn": (_I, [_P, _P, _I, _P, _L, _P, _P, _P, _L, _I, _I, _I, _I, _F, _I, _P, _I, _P]),
+    "b200_seq_latent_attn": (_I, [_P, _P, _I, _P, _L, _P, _P, _P, _L, _I, _I, _I, _I, _F, _I, _P, _I, _P, _P]),
     "b200_seq_causal_conv_silu": (_I, [_P, _L, _I, _I, _I, _P, _P, _I, _P, _P, _P, _P, _P, _P, _L, _I, _P]),
     "b200_seq_ssm_scan": (_I, [_P, _L, _I, _I, _I, _P, _L, _I, _P, _P, _P, _I, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P]),
     "b200_seq_mlstm_scan": (_I, [_P, _L, _I, _I, _I, _I, _I, _P, _P, _I, _F, _F, _P, _P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _P]),
@@ -151,10 +151,11 @@ SEQ_SIGNATURES = {
     "b200_seq_diff_combine": (_I, [_P, _P, _I, _L, _I, _I, _F, _F, _F, _P]),
     "b200_seq_moe_plan_ints": (_L, [_L, _I, _I]),
     "b200_seq_moe_route": (_I, [_P, _L, _I, _I, _P, _P, _P, _P]),
-    "b200_seq_moe_linear": (_I, [_P, _I, _L, _I, _P, _I, _P, _I, _L, _P, _L, _I, _I, _L, _L, _P]),
+    "b200_seq_moe_linear": (_I, [_P, _I, _L, _I, _P, _I, _P, _I, _L, _P, _L, _I, _I, _L, _L, _I, _P]),
     "b200_seq_moe_gather_rows": (_I, [_P, _I, _L, _P, _P, _L, _I, _I, _L, _P]),
     "b200_seq_moe_combine_add": (_I, [_P, _P, _P, _L, _P, _P, _L, _I, _I, _L, _P]),
-    "b200_seq_moe_route_scored": (_I, [_P, _L, _I, _I, _I, _P, _I, _F, _P, _P, _P, _P]),
+    "b200_seq_moe_route_scored": (_I, [_P, _L, _L, _I, _I, _I, _I, _P, _I, _F, _P, _P, _P, _P]),
+    "b200_seq_moe_row_of": (_P, [_P, _L, _I, _I]),
     "b200_seq_gated_rms_add": (_I, [_P, _P, _P, _I, _P, _P, _L, _L, _F, _P]),
     "b200_seq_cast_rows": (_I, [_P, _P, _I, _L, _P]),
     "b200_seq_ff_gate": (_I, [_P, _P, _I, _L, _L, _I, _P]),
@@ -164,10 +165,12 @@ SEQ_SIGNATURES = {
                                     _P]),
     "b200_seq_delta_rows_scan": (_I, [_P, _I, _P, _P, _P, _P, _P, _L, _L, _I, _I, _I, _I, _I, _P]),
     "b200_seq_qk_rot_prepare": (_I, [_P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _P, _I, _F, _P, _P, _I, _P, _P, _P, _I, _L, _I, _I, _P, _L, _P, _P, _I,
-                                     _I, _P]),
+                                     _I, _I, _P]),
     "b200_seq_talk_attn": (_I, [_P, _P, _I, _L, _I, _I, _P, _L, _P, _P, _I, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _P]),
     "b200_seq_streams_step": (_I, [_P, _I, _P, _P, _P, _P, _P, _P, _I, _P, _L, _L, _F, _P]),
     "b200_seq_branches_step": (_I, [_P, _P, _P, _P, _P, _P, _F, _P, _P, _P, _I, _P, _L, _L, _F, _P]),
+    "b200_seq_halves_step": (_I, [_P, _P, _P, _P, _P, _L, _P, _L, _P, _P, _I, _P, _P, _P, _I, _P, _P, _L, _L, _F, _P]),
+    "b200_seq_soft_cap": (_I, [_P, _L, _F, _P]),
     "b200_seq_ff_act": (_I, [_P, _I, _L, _P, _I, _L, _L, _I, _P]),
     "b200_seq_heads_turn_gate": (_I, [_P, _P, _L, _P, _P, _I, _I, _P, _P, _I, _L, _F, _L, _I, _I, _P]),
     "b200_seq_gdelta_scan": (_I, [_P, _L, _I, _I, _I, _I, _P, _L, _I, _P, _P, _I, _F, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _P]),

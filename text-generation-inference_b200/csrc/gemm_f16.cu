@@ -21,7 +21,7 @@ namespace b200 {
 
 // Element formats of one instantiation: 0 = fp16 operands, fp16 output (the flash families); 1 = bfloat16 operands, bfloat16
 // output; 2 = bfloat16 operands, fp32 output (hybrid families: projections whose results enter a recurrence, a norm or the
-// soft-max stay in 32 bits).  Same pipeline; the instruction descriptor's operand formats and the epilogue's stores differ.
+// soft-max stay in 32 bits); 3 = as 1 with the square of ReLU on the result.  Same pipeline; the instruction descriptor's operand formats and the epilogue's stores differ.
 template <int FMT>
 __device__ __forceinline__ float gemm_load_bias(const void* bias, int n) {
   if constexpr (FMT == 0) return __half2float(reinterpret_cast<const __half*>(bias)[n]);
@@ -31,6 +31,7 @@ template <int FMT>
 __device__ __forceinline__ void gemm_store(void* y, size_t i, float v) {
   if constexpr (FMT == 0) reinterpret_cast<__half*>(y)[i] = __float2half_rn(v);
   else if constexpr (FMT == 1) reinterpret_cast<__nv_bfloat16*>(y)[i] = __float2bfloat16_rn(v);
+  else if constexpr (FMT == 3) reinterpret_cast<__nv_bfloat16*>(y)[i] = __float2bfloat16_rn(v < 0.f ? 0.f : v * v);
   else reinterpret_cast<float*>(y)[i] = v;
 }
 
@@ -449,11 +450,12 @@ extern "C" int b200_gemm_f16(const void* x, const void* w, const void* bias, voi
                              void* workspace, void* stream) {
   return gemm_f16_impl<0>(x, w, bias, y, T, N, K, workspace, nullptr, stream);
 }
-// bfloat16 x [T, K] and w [N, K] (bias bfloat16 or NULL) -> y [T, N] bfloat16, or fp32 when out_f32 != 0.  Same kernel,
-// workspace and rules as b200_gemm_f16.
-extern "C" int b200_gemm_bf16(const void* x, const void* w, const void* bias, void* y, int out_f32, int64_t T, int64_t N, int64_t K,
+// bfloat16 x [T, K] and w [N, K] (bias bfloat16 or NULL) -> y [T, N]; out_kind 0: bfloat16, 1: fp32, 2: bfloat16 after the square of
+// ReLU.  Same kernel, workspace and rules as b200_gemm_f16.
+extern "C" int b200_gemm_bf16(const void* x, const void* w, const void* bias, void* y, int out_kind, int64_t T, int64_t N, int64_t K,
                               void* workspace, void* stream) {
-  if (out_f32) return gemm_f16_impl<2>(x, w, bias, y, T, N, K, workspace, nullptr, stream);
+  if (out_kind == 2) return gemm_f16_impl<3>(x, w, bias, y, T, N, K, workspace, nullptr, stream);
+  if (out_kind == 1) return gemm_f16_impl<2>(x, w, bias, y, T, N, K, workspace, nullptr, stream);
   return gemm_f16_impl<1>(x, w, bias, y, T, N, K, workspace, nullptr, stream);
 }
 extern "C" int b200_gemm_f16_deferred(const void* x, const void* w, const void* bias, int64_t T, int64_t N, int64_t K, void* workspace,

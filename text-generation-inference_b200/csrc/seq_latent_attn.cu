@@ -79,7 +79,7 @@ template <typename T, int NR>
 __global__ void __launch_bounds__(kHeadsPerBlock * 32) latent_attn_kernel(
     const float* __restrict__ q_abs, const T* __restrict__ cache, const int32_t* __restrict__ block_table, int64_t bt_stride,
     const int32_t* __restrict__ seq_of_token, const int64_t* __restrict__ position_ids, float* __restrict__ out, int H, int R, int D, int window,
-    float scale, int page) {
+    float scale, int page, const float* __restrict__ sink) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float sm[];
@@ -97,7 +97,8 @@ __global__ void __launch_bounds__(kHeadsPerBlock * 32) latent_attn_kernel(
     const int hh = h0 + idx / D;
     qs[idx] = hh < H ? q_abs[(t * H + hh) * D + idx % D] : 0.f;
   }
-  float m = -INFINITY, l = 0.f;
+  // a sink logit sits in the soft-max denominator like one more key (unscaled) whose value is zero
+  float m = (sink && h < H) ? sink[h] : -INFINITY, l = (sink && h < H) ? 1.f : 0.f;
   float acc[NR];
 #pragma unroll
   for (int i = 0; i < NR; ++i) acc[i] = 0.f;
@@ -164,7 +165,7 @@ template <int NTW>  // n-tiles (8 output columns each) per warp: R = 32 * NTW
 __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(
     const float* __restrict__ q_abs, const __nv_bfloat16* __restrict__ cache, const int32_t* __restrict__ block_table, int64_t bt_stride,
     const int32_t* __restrict__ seq_of_token, const int64_t* __restrict__ position_ids, float* __restrict__ out, int H, int R, int D, int window,
-    float scale, int page, float* __restrict__ partial) {
+    float scale, int page, float* __restrict__ partial, const float* __restrict__ sink) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -195,6 +196,14 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(
   }
   const int r0 = lane >> 2, cq = (lane & 3) * 2;   // accumulator rows r0, r0 + 8; columns cq, cq + 1 of an 8-wide tile
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+  if (sink && blockIdx.z == 0) {   // the sink counts once: in the first run of the keys
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+      if (h0 + r0 + i * 8 < H) {
+        m_run[i] = sink[h0 + r0 + i * 8];
+        l_run[i] = 1.f;
+      }
+  }
   float o[NTW][4];
 #pragma unroll
   for (int i = 0; i < NTW; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
@@ -402,14 +411,14 @@ extern "C" int b200_seq_latent_prepare(const float* down, int64_t ld_down, int c
 template <typename T, int NR>
 static int launch_latent_attn(const float* q_abs, const void* cache, const int32_t* block_table, int64_t bt_stride, const int32_t* seq_of_token,
                               const int64_t* position_ids, float* out, int64_t Tq, int H, int R, int D, int window, float scale, int page,
-                              cudaStream_t st) {
+                              const float* sink, cudaStream_t st) {
   const size_t smem = ((size_t)kHeadsPerBlock * D + (size_t)kKeyTile * (D + 1)) * 4;
   if (smem > 200 * 1024) { b200_set_last_error("seq_latent_attn: cache row too wide"); return B200_ERR_ARG; }
   static bool cfg = false;
   if (!cfg) { cudaFuncSetAttribute(latent_attn_kernel<T, NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); cfg = true; }
   dim3 grid((unsigned)Tq, (unsigned)((H + kHeadsPerBlock - 1) / kHeadsPerBlock));
   B200_LAUNCH((latent_attn_kernel<T, NR>), grid, dim3(kHeadsPerBlock * 32), smem, st, q_abs, (const T*)cache, block_table, bt_stride, seq_of_token,
-              position_ids, out, H, R, D, window, scale, page);
+              position_ids, out, H, R, D, window, scale, page, sink);
   b200_count_launches(1);
   return B200_OK;
 }
@@ -428,10 +437,11 @@ extern "C" int b200_seq_latent_attn_splits(int dt, int64_t Tq, int H, int R, int
   return (int)n;
 }
 
-// `partial` / nsplit: from b200_seq_latent_attn_splits (NULL / <= 1: no split).
+// `partial` / nsplit: from b200_seq_latent_attn_splits (NULL / <= 1: no split).  sink fp32 [H] or NULL: a logit per head that joins
+// the soft-max denominator (unscaled) and carries no value.
 extern "C" int b200_seq_latent_attn(const float* q_abs, const void* cache, int dt, const int32_t* block_table, int64_t bt_stride,
                                     const int32_t* seq_of_token, const int64_t* position_ids, float* out, int64_t Tq, int H, int R, int r,
-                                    int window, float scale, int page, float* partial, int nsplit, void* stream) {
+                                    int window, float scale, int page, float* partial, int nsplit, const float* sink, void* stream) {
   if (Tq == 0) return B200_OK;
   const int D = R + r;
   if (window <= 0) window = 0x3fffffff;
@@ -448,7 +458,7 @@ extern "C" int b200_seq_latent_attn(const float* q_abs, const void* cache, int d
     static bool cfg = false;                                                                                                          \
     if (!cfg) { cudaFuncSetAttribute(latent_attn_mma_kernel<N>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); cfg = true; } \
     B200_LAUNCH((latent_attn_mma_kernel<N>), grid, dim3(kMmaThreads), smem, st, q_abs, (const __nv_bfloat16*)cache, block_table, bt_stride, \
-                seq_of_token, position_ids, out, H, R, D, window, scale, page, partial);                                              \
+                seq_of_token, position_ids, out, H, R, D, window, scale, page, partial, sink);                                              \
     if (nsplit > 1)                                                                                                                   \
       B200_LAUNCH(latent_attn_merge_kernel, dim3((unsigned)((Tq * H + 3) / 4)), dim3(128), 0, st, (const float*)partial, out, Tq, H, R, \
                   (int)grid.y, nsplit);                                                                                              \
@@ -470,7 +480,7 @@ extern "C" int b200_seq_latent_attn(const float* q_abs, const void* cache, int d
   }
 #define LA(NR)                                                                                                                         \
   B200_SEQ_DISPATCH(dt, E, return (launch_latent_attn<E, NR>(q_abs, cache, block_table, bt_stride, seq_of_token, position_ids, out, Tq, H, R, D, \
-                                                            window, scale, page, st)))
+                                                            window, scale, page, sink, st)))
   if (nr <= 4) LA(4);
   else if (nr <= 8) LA(8);
   else if (nr <= 16) LA(16);

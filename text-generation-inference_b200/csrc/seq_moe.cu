@@ -1,16 +1,21 @@
-// Routed feed-forward (mixture of experts): every token picks `top` experts and weighs them, by one of two rules:
+// Routed feed-forward (mixture of experts): every token picks `top` experts and weighs them, by one of three rules:
 //   mode 0  the largest router logits; weights = soft-max over the picked logits only;
 //   mode 1  scores s = sigmoid(logit); the largest s + correction[expert] are picked, the weights are the picked plain scores
-//           divided by their sum (+ 1e-20), times a constant.
+//           divided by their sum (+ 1e-20), times a constant;
+//   mode 2  as mode 1 with s = soft-max of the logits over all router outputs.
+// The last router outputs may be identity outputs (no tensors: their result is the token's input): they take no row of the plan, and
+// row_of is -1 for such a pick.
 //
 //   moe_route_kernel   : one warp per token: top-k of the fp32 logits (ties: the lower expert), weights, and the token's place in
-//                        each picked expert's list (an atomic counter per expert; the order inside a list changes no result).
+//                        each picked expert's list (an atomic counter per expert; the order inside a list changes no result);
+//                        moe_route_plan_kernel does this and the plan in one launch for a step of few tokens.
 //   moe_plan_kernel    : lists -> one compact row order (expert by expert) cut into tiles of 64 rows that never span two
 //                        experts; row <-> (token, pick) maps in both directions.
 //   moe_linear_kernel  : C[row] = W[expert of row's tile] A[row] over that plan; A rows are either the compact rows or gathered
 //                        through the row -> token map.  fp32 accumulation in ascending k: a row's result does not depend on what
 //                        else the step holds.
 //   moe_linear_mma_kernel : the same product on tensor cores for bfloat16 operands (see the note above the kernel).
+//                        Both may end with the square of ReLU on the product (act 1).
 //   moe_combine_add_kernel : resid[t] += mix[t] + sum over the token's picks, in pick order, of weight * y[row(t, pick)].
 //
 // Plan workspace (int32): [counts E][offsets E + 1][n_tiles 1][tile_expert max_tiles][tile_row0 max_tiles][place R][row_of R]
@@ -46,24 +51,38 @@ __host__ __device__ inline MoePlan moe_plan_view(int32_t* base, int64_t T, int E
   return p;
 }
 
-template <int MODE>
-__global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict__ logits, int64_t T, int E, int top, int32_t* __restrict__ ids,
-                                                        float* __restrict__ weights, int32_t* __restrict__ counts, int32_t* __restrict__ place,
-                                                        const void* __restrict__ correction, int corr_dt, float weight_scale) {
-  pdl_launch_dependents();
-  pdl_wait();
-  const int64_t t = (int64_t)blockIdx.x * 8 + warp_id();
-  if (t >= T) return;
+// One warp: the `top` picks of one token from its E router outputs (fp32) and their weights; `took(k, e)` runs in lane 0 for every pick
+template <int MODE, typename Took>
+__device__ __forceinline__ void moe_pick(const float* __restrict__ row, int E, int top, const void* __restrict__ correction, int corr_dt,
+                                         float weight_scale, float* __restrict__ w_out, Took took) {
   const int lane = lane_id();
   float z[kMaxExpertsPerLane], sc[kMaxExpertsPerLane];
 #pragma unroll
   for (int i = 0; i < kMaxExpertsPerLane; ++i) {
     const int e = lane + 32 * i;
-    z[i] = e < E ? logits[t * E + e] : -INFINITY;
+    z[i] = e < E ? row[e] : -INFINITY;
     sc[i] = 0.f;
-    if (MODE == 1 && e < E) {
-      sc[i] = sigmoid_f(z[i]);
-      z[i] = sc[i] + (correction ? ld_any(correction, e, corr_dt) : 0.f);
+    if (MODE == 1 && e < E) sc[i] = sigmoid_f(z[i]);
+  }
+  if (MODE == 2) {  // soft-max over all router outputs
+    float m = z[0], sum = 0.f;
+#pragma unroll
+    for (int i = 1; i < kMaxExpertsPerLane; ++i) m = fmaxf(m, z[i]);
+    m = warp_max(m);
+#pragma unroll
+    for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+      sc[i] = lane + 32 * i < E ? expf(z[i] - m) : 0.f;
+      sum += sc[i];
+    }
+    const float inv = 1.f / warp_sum(sum);
+#pragma unroll
+    for (int i = 0; i < kMaxExpertsPerLane; ++i) sc[i] *= inv;
+  }
+  if (MODE != 0) {
+#pragma unroll
+    for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+      const int e = lane + 32 * i;
+      if (e < E) z[i] = sc[i] + (correction ? ld_any(correction, e, corr_dt) : 0.f);
     }
   }
   float val[kMaxTop];
@@ -84,7 +103,8 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict_
       const int oe = __shfl_xor_sync(0xffffffffu, be, o);
       if (ov > best || (ov == best && oe < be)) { best = ov; be = oe; }
     }
-    if (MODE == 1) {  // the weight uses the plain score of the pick, which its owning lane holds
+    if (be >= E) be = 0;  // only when no comparison held (logits that are not numbers): stay in bounds
+    if (MODE != 0) {  // the weight uses the plain score of the pick, which its owning lane holds
       float mine = 0.f;
 #pragma unroll
       for (int i = 0; i < kMaxExpertsPerLane; ++i)
@@ -102,49 +122,125 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict_
 #pragma unroll
     for (int k = 0; k < kMaxTop; ++k) {
       if (k >= top) break;
-      w[k] = MODE == 1 ? val[k] : expf(val[k] - val[0]);  // mode 0: val[0] is the largest
+      w[k] = MODE != 0 ? val[k] : expf(val[k] - val[0]);  // mode 0: val[0] is the largest
       den += w[k];
     }
-    const float norm = MODE == 1 ? weight_scale / (den + 1e-20f) : 1.f / den;
+    const float norm = MODE != 0 ? weight_scale / (den + 1e-20f) : 1.f / den;
 #pragma unroll
     for (int k = 0; k < kMaxTop; ++k) {
       if (k >= top) break;
-      ids[t * top + k] = idx[k];
-      weights[t * top + k] = w[k] * norm;
-      place[t * top + k] = atomicAdd(counts + idx[k], 1);
+      w_out[k] = w[k] * norm;
+      took(k, idx[k]);
     }
   }
 }
 
-__global__ void __launch_bounds__(256) moe_plan_kernel(const int32_t* __restrict__ ids, int64_t R, int top, int E, MoePlan p) {
-  pdl_launch_dependents();
-  pdl_wait();
-  if (threadIdx.x == 0) {
-    int off = 0, nt = 0;
-    for (int e = 0; e < E; ++e) {
-      p.offsets[e] = off;
-      const int c = p.counts[e];
-      for (int r = 0; r < c; r += kMoeTile) {
-        p.tile_expert[nt] = e;
-        p.tile_row0[nt] = off + r;
-        ++nt;
-      }
-      off += c;
+// The plan from the experts' counts (a block, counts in shared memory): row offsets and tiles of every expert.  `offs` [E + 1] receives
+// the offsets as well.  The first 32 threads scan 8 experts each.
+__device__ __forceinline__ void moe_offsets(const int* counts, int* offs, int E, const MoePlan& p) {
+  if (threadIdx.x < 32) {
+    int c[kMaxExpertsPerLane], rows = 0, tiles = 0;
+#pragma unroll
+    for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+      const int e = threadIdx.x * kMaxExpertsPerLane + i;
+      c[i] = e < E ? counts[e] : 0;
+      rows += c[i];
+      tiles += (c[i] + kMoeTile - 1) / kMoeTile;
     }
-    p.offsets[E] = off;
-    *p.n_tiles = nt;
+    int r0 = rows, t0 = tiles;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int r = __shfl_up_sync(0xffffffffu, r0, o), t = __shfl_up_sync(0xffffffffu, t0, o);
+      if ((int)threadIdx.x >= o) { r0 += r; t0 += t; }
+    }
+    if (threadIdx.x == 31) {
+      offs[E] = r0;
+      p.offsets[E] = r0;
+      *p.n_tiles = t0;
+    }
+    r0 -= rows;
+    t0 -= tiles;
+#pragma unroll
+    for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+      const int e = threadIdx.x * kMaxExpertsPerLane + i;
+      if (e >= E) break;
+      offs[e] = r0;
+      p.offsets[e] = r0;
+      for (int r = 0; r < c[i]; r += kMoeTile) {
+        p.tile_expert[t0] = e;
+        p.tile_row0[t0] = r0 + r;
+        ++t0;
+      }
+      r0 += c[i];
+    }
   }
   __syncthreads();
+}
+
+// picks of the whole step, 8 tokens per block; the places in the experts' lists come from counters in the plan.  Router outputs from E
+// on (up to E_all) are identity outputs: they are picked like experts but take no row (place -1).
+template <int MODE>
+__global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict__ logits, int64_t ld, int64_t T, int E, int E_all, int top,
+                                                        int32_t* __restrict__ ids, float* __restrict__ weights, MoePlan p,
+                                                        const void* __restrict__ correction, int corr_dt, float weight_scale) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t t = (int64_t)blockIdx.x * 8 + warp_id();
+  if (t >= T) return;
+  moe_pick<MODE>(logits + t * ld, E_all, top, correction, corr_dt, weight_scale, weights + t * top, [&](int k, int e) {
+    ids[t * top + k] = e;
+    p.place[t * top + k] = e < E ? atomicAdd(p.counts + e, 1) : -1;
+  });
+}
+
+__global__ void __launch_bounds__(1024) moe_plan_kernel(const int32_t* __restrict__ ids, int64_t R, int top, int E, MoePlan p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ int counts[32 * kMaxExpertsPerLane], offs[32 * kMaxExpertsPerLane + 1];
+  for (int e = threadIdx.x; e < E; e += blockDim.x) counts[e] = p.counts[e];
+  __syncthreads();
+  moe_offsets(counts, offs, E, p);
   for (int64_t i = threadIdx.x; i < R; i += blockDim.x) {
-    const int row = p.offsets[ids[i]] + p.place[i];
+    const int e = ids[i];
+    const int row = e < E ? offs[e] + p.place[i] : -1;
     p.row_of[i] = row;
-    p.token_of_row[row] = (int32_t)(i / top);
+    if (row >= 0) p.token_of_row[row] = (int32_t)(i / top);
   }
 }
+
+// picks and plan of a step of few tokens (decoding) in one launch: one block, counters in shared memory
+constexpr int kRouteOnePass = 64;
+
+template <int MODE>
+__global__ void __launch_bounds__(1024) moe_route_plan_kernel(const float* __restrict__ logits, int64_t ld, int T, int E, int E_all, int top,
+                                                              int32_t* __restrict__ ids, float* __restrict__ weights, MoePlan p,
+                                                              const void* __restrict__ correction, int corr_dt, float weight_scale) {
+  pdl_launch_dependents();
+  __shared__ int counts[32 * kMaxExpertsPerLane], offs[32 * kMaxExpertsPerLane + 1];
+  __shared__ int s_id[kRouteOnePass * kMaxTop], s_place[kRouteOnePass * kMaxTop];
+  for (int e = threadIdx.x; e < E; e += blockDim.x) counts[e] = 0;
+  __syncthreads();
+  pdl_wait();
+  for (int t = warp_id(); t < T; t += blockDim.x / 32)
+    moe_pick<MODE>(logits + t * ld, E_all, top, correction, corr_dt, weight_scale, weights + t * top, [&](int k, int e) {
+      s_id[t * top + k] = e;
+      s_place[t * top + k] = e < E ? atomicAdd(counts + e, 1) : -1;
+    });
+  __syncthreads();
+  moe_offsets(counts, offs, E, p);
+  for (int i = threadIdx.x; i < T * top; i += blockDim.x) {
+    const int e = s_id[i], row = e < E ? offs[e] + s_place[i] : -1;
+    ids[i] = e;
+    p.row_of[i] = row;
+    if (row >= 0) p.token_of_row[row] = i / top;
+  }
+}
+
+__device__ __forceinline__ float moe_act(float v, int act) { return act == 1 ? (v < 0.f ? 0.f : v * v) : v; }
 
 template <typename TA, typename TW, typename TC>
 __global__ void __launch_bounds__(256) moe_linear_kernel(const TA* __restrict__ A, int64_t lda, int gather, const TW* __restrict__ W,
-                                                         TC* __restrict__ C, int64_t ldc, MoePlan p, int N, int K) {
+                                                         TC* __restrict__ C, int64_t ldc, MoePlan p, int N, int K, int act) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float As[kMoeStep][kMoeTile + 4];
@@ -195,7 +291,7 @@ __global__ void __launch_bounds__(256) moe_linear_kernel(const TA* __restrict__ 
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
-      if (n < N) stf(C + (int64_t)m * ldc + n, acc[i][j]);
+      if (n < N) stf(C + (int64_t)m * ldc + n, moe_act(acc[i][j], act));
     }
   }
 }
@@ -209,7 +305,7 @@ constexpr int kMmaBK = 64, kMmaStages = 3, kMmaLd = kMmaBK + 8;
 template <typename TC>
 __global__ void __launch_bounds__(128) moe_linear_mma_kernel(const __nv_bfloat16* __restrict__ A, int64_t lda, int gather,
                                                              const __nv_bfloat16* __restrict__ W, TC* __restrict__ C, int64_t ldc, MoePlan p, int N,
-                                                             int K) {
+                                                             int K, int act) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) unsigned char moe_smem[];
@@ -282,17 +378,18 @@ __global__ void __launch_bounds__(128) moe_linear_mma_kernel(const __nv_bfloat16
       for (int el = 0; el < 4; ++el) {
         const int m = m0 + wm * 32 + mt * 16 + (lane >> 2) + (el >> 1) * 8;
         const int n = n0 + wn * 32 + nt * 8 + cq + (el & 1);
-        if (m < m_end && n < N) stf(C + (int64_t)m * ldc + n, acc[mt][nt][el]);
+        if (m < m_end && n < N) stf(C + (int64_t)m * ldc + n, moe_act(acc[mt][nt][el], act));
       }
 }
 
 // out[row] = A[token(row)] for the compact rows of the plan (what a dense product per expert reads)
 template <typename T>
 __global__ void __launch_bounds__(256) moe_gather_rows_kernel(const T* __restrict__ A, int64_t lda, T* __restrict__ out, const int32_t* __restrict__ token_of_row,
-                                                              int K) {
+                                                              const int32_t* __restrict__ n_rows, int K) {
   pdl_launch_dependents();
   pdl_wait();
   const int64_t row = blockIdx.x;
+  if (row >= *n_rows) return;   // picks of identity outputs have no row
   const T* src = A + (int64_t)token_of_row[row] * lda;
   for (int i = threadIdx.x; i < K; i += 256) out[row * K + i] = src[i];
 }
@@ -320,46 +417,58 @@ extern "C" int64_t b200_seq_moe_plan_ints(int64_t T, int E, int top) {
   return (int64_t)E + E + 1 + 1 + 2 * moe_max_tiles(T, E, top) + 3 * T * top;
 }
 
-// logits fp32 [T, E] -> ids int32 [T, top], weights fp32 [T, top] and the plan (b200_seq_moe_plan_ints int32 values)
-// mode 0: soft-max over the picked logits (correction, weight_scale unused); mode 1: sigmoid scores, picks by score + correction
-// (element type corr_dt, may be NULL), weights = score / sum of the picked scores * weight_scale
-extern "C" int b200_seq_moe_route_scored(const float* logits, int64_t T, int E, int top, int mode, const void* correction, int corr_dt,
-                                         float weight_scale, int32_t* ids, float* weights, int32_t* plan, void* stream) {
+extern "C" int32_t* b200_seq_moe_row_of(int32_t* plan, int64_t T, int E, int top) { return moe_plan_view(plan, T, E, top).row_of; }
+
+// logits fp32 [T, E_all] (leading dimension ld) -> ids int32 [T, top], weights fp32 [T, top] and the plan (b200_seq_moe_plan_ints(T, E, top)
+// int32 values) over the E experts; the router outputs E .. E_all - 1 are identity outputs.
+// mode 0: soft-max over the picked logits (correction, weight_scale unused); mode 1 / 2: scores sigmoid(logit) / soft-max over all E_all
+// outputs, picks by score + correction (element type corr_dt, may be NULL), weights = score / sum of the picked scores * weight_scale
+extern "C" int b200_seq_moe_route_scored(const float* logits, int64_t ld, int64_t T, int E, int E_all, int top, int mode, const void* correction,
+                                         int corr_dt, float weight_scale, int32_t* ids, float* weights, int32_t* plan, void* stream) {
   if (T == 0) return B200_OK;
-  if (E < 1 || E > 32 * kMaxExpertsPerLane || top < 1 || top > kMaxTop || top > E) {
-    b200_set_last_error("seq_moe_route: need 1 <= top <= min(16, experts), experts <= 256");
+  if (E < 1 || E_all < E || E_all > 32 * kMaxExpertsPerLane || top < 1 || top > kMaxTop || top > E_all || mode < 0 || mode > 2 || ld < E_all) {
+    b200_set_last_error("seq_moe_route: need 1 <= top <= min(16, router outputs), 1 <= experts <= router outputs <= 256");
     return B200_ERR_ARG;
   }
   cudaStream_t st = (cudaStream_t)stream;
   MoePlan p = moe_plan_view(plan, T, E, top);
-  if (cudaMemsetAsync(p.counts, 0, sizeof(int32_t) * E, st) != cudaSuccess) { b200_set_last_error("seq_moe_route: memset failed"); return B200_ERR_CUDA; }
-  if (mode == 1)
-    B200_LAUNCH(moe_route_kernel<1>, dim3((unsigned)((T + 7) / 8)), dim3(256), 0, st, logits, T, E, top, ids, weights, p.counts, p.place, correction,
-                corr_dt, weight_scale);
-  else
-    B200_LAUNCH(moe_route_kernel<0>, dim3((unsigned)((T + 7) / 8)), dim3(256), 0, st, logits, T, E, top, ids, weights, p.counts, p.place, correction,
-                corr_dt, weight_scale);
-  B200_LAUNCH(moe_plan_kernel, dim3(1), dim3(256), 0, st, (const int32_t*)ids, T * top, top, E, p);
+#define ROUTE(M)                                                                                                                          \
+  do {                                                                                                                                    \
+    if (T <= kRouteOnePass) {                                                                                                             \
+      B200_LAUNCH(moe_route_plan_kernel<M>, dim3(1), dim3(T <= 8 ? 256 : 1024), 0, st, logits, ld, (int)T, E, E_all, top, ids, weights, p, \
+                  correction, corr_dt, weight_scale);                                                                                     \
+      b200_count_launches(1);                                                                                                             \
+      return B200_OK;                                                                                                                     \
+    }                                                                                                                                     \
+    if (cudaMemsetAsync(p.counts, 0, sizeof(int32_t) * E, st) != cudaSuccess) { b200_set_last_error("seq_moe_route: memset failed"); return B200_ERR_CUDA; } \
+    B200_LAUNCH(moe_route_kernel<M>, dim3((unsigned)((T + 7) / 8)), dim3(256), 0, st, logits, ld, T, E, E_all, top, ids, weights, p, correction, \
+                corr_dt, weight_scale);                                                                                                   \
+  } while (0)
+  if (mode == 2) ROUTE(2);
+  else if (mode == 1) ROUTE(1);
+  else ROUTE(0);
+#undef ROUTE
+  B200_LAUNCH(moe_plan_kernel, dim3(1), dim3(1024), 0, st, (const int32_t*)ids, T * top, top, E, p);
   b200_count_launches(2);
   return B200_OK;
 }
 
 extern "C" int b200_seq_moe_route(const float* logits, int64_t T, int E, int top, int32_t* ids, float* weights, int32_t* plan, void* stream) {
-  return b200_seq_moe_route_scored(logits, T, E, top, 0, nullptr, B200_DT_F32, 1.f, ids, weights, plan, stream);
+  return b200_seq_moe_route_scored(logits, E, T, E, E, top, 0, nullptr, B200_DT_F32, 1.f, ids, weights, plan, stream);
 }
 
 template <typename TA, typename TW, typename TC>
 static int launch_moe_linear(const void* A, int64_t lda, int gather, const void* W, void* C, int64_t ldc, MoePlan p, int64_t N, int64_t K,
-                             cudaStream_t st) {
+                             int act, cudaStream_t st) {
   dim3 grid((unsigned)((N + kMoeTile - 1) / kMoeTile), (unsigned)p.max_tiles);
-  B200_LAUNCH((moe_linear_kernel<TA, TW, TC>), grid, dim3(256), 0, st, (const TA*)A, lda, gather, (const TW*)W, (TC*)C, ldc, p, (int)N, (int)K);
+  B200_LAUNCH((moe_linear_kernel<TA, TW, TC>), grid, dim3(256), 0, st, (const TA*)A, lda, gather, (const TW*)W, (TC*)C, ldc, p, (int)N, (int)K, act);
   b200_count_launches(1);
   return B200_OK;
 }
 
-// C[row, :N] = W[expert(row)] [N, K] . A[gather ? token(row) : row, :K] for the T * top compact rows of the plan; W [E, N, K] dense
+// act 0: none, 1: the square of ReLU.  C[row, :N] = act(W[expert(row)] [N, K] . A[gather ? token(row) : row, :K]) for the T * top compact rows of the plan; W [E, N, K] dense
 extern "C" int b200_seq_moe_linear(const void* A, int a_dt, int64_t lda, int gather, const void* W, int w_dt, void* C, int c_dt, int64_t ldc,
-                                   int32_t* plan, int64_t T, int E, int top, int64_t N, int64_t K, void* stream) {
+                                   int32_t* plan, int64_t T, int E, int top, int64_t N, int64_t K, int act, void* stream) {
   if (T == 0 || N == 0) return B200_OK;
   MoePlan p = moe_plan_view(plan, T, E, top);
   if (p.max_tiles > 65535 || K <= 0) { b200_set_last_error("seq_moe_linear: bad sizes"); return B200_ERR_ARG; }
@@ -374,7 +483,7 @@ extern "C" int b200_seq_moe_linear(const void* A, int a_dt, int64_t lda, int gat
     static bool cfg = false;                                                                                                            \
     if (!cfg) { cudaFuncSetAttribute(moe_linear_mma_kernel<TC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); cfg = true; }   \
     B200_LAUNCH((moe_linear_mma_kernel<TC>), grid, dim3(128), smem, st, (const __nv_bfloat16*)A, lda, gather, (const __nv_bfloat16*)W,   \
-                (TC*)C, ldc, p, (int)N, (int)K);                                                                                        \
+                (TC*)C, ldc, p, (int)N, (int)K, act);                                                                                   \
     b200_count_launches(1);                                                                                                             \
     return B200_OK;                                                                                                                     \
   } while (0)
@@ -384,7 +493,7 @@ extern "C" int b200_seq_moe_linear(const void* A, int a_dt, int64_t lda, int gat
   }
   const int key = a_dt * 4 + w_dt * 2 + c_dt;
 #define CASE(a, w, c, TA, TW, TC) \
-  case a * 4 + w * 2 + c: return launch_moe_linear<TA, TW, TC>(A, lda, gather, W, C, ldc, p, N, K, st)
+  case a * 4 + w * 2 + c: return launch_moe_linear<TA, TW, TC>(A, lda, gather, W, C, ldc, p, N, K, act, st)
   switch (key) {
     CASE(0, 0, 0, __nv_bfloat16, __nv_bfloat16, __nv_bfloat16);
     CASE(0, 0, 1, __nv_bfloat16, __nv_bfloat16, float);
@@ -415,7 +524,7 @@ extern "C" int b200_seq_moe_gather_rows(const void* A, int dt, int64_t lda, void
   if (T == 0) return B200_OK;
   MoePlan p = moe_plan_view(plan, T, E, top);
   B200_SEQ_DISPATCH(dt, El, B200_LAUNCH((moe_gather_rows_kernel<El>), dim3((unsigned)(T * top)), dim3(256), 0, (cudaStream_t)stream, (const El*)A, lda,
-                                        (El*)out, (const int32_t*)p.token_of_row, (int)K));
+                                        (El*)out, (const int32_t*)p.token_of_row, (const int32_t*)(p.offsets + E), (int)K));
   b200_count_launches(1);
   return B200_OK;
 }

@@ -2,7 +2,8 @@
 // the stream, RMS norm of the stream with an offset weight, RMS norm of a
 // column slice, grouped RMS norm with a gate, the clamped gated feed-forward activation, the per-layer token side input, the step
 // between two sublayers of a decoder with several residual streams (write all streams, read and norm the next input) and of one
-// whose sublayers have one or two branches, each with a norm of its own, plain activations, and the turn-back + gate of attention heads whose values carry their position.
+// whose sublayers have one or two branches, each with a norm of its own, the step between two layers that add a mixer and a routed
+// feed-forward side by side, the soft cap on logits, plain activations, and the turn-back + gate of attention heads whose values carry their position.
 // One block per token row; all statistics and the residual sum in fp32.
 #include "seq_common.cuh"
 
@@ -412,6 +413,99 @@ __global__ void __launch_bounds__(kRowThreads) branches_step_kernel(float* __res
   }
 }
 
+// One stream whose layers read it once and add two halves side by side (row t of x, fp32): what lies between two layers in one launch,
+//   r = (init ? init[t] : x[t]) + y1[t] + sigmoid(gate[t]) * y2[t] + sum_k weights[t, k] * (row_of[t, k] >= 0 ? rows[row_of[t, k]] : pass[t]),
+//   x[t] <- r, typed_a[t] <- n(r) * norm_a, typed_b[t] <- n(r) * norm_b with n(r) = r / sqrt(mean(r^2) + eps)
+// (any term may be missing, gate NULL: y2 as it is).  The sum is a routed feed-forward's: experts' rows, and for a pick of an identity
+// output the row `pass` that the router read.  One block per token; r waits in shared memory between the passes.
+constexpr int kPicks = 16;
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kRowThreads) halves_step_kernel(float* __restrict__ x, const float* __restrict__ init, const float* __restrict__ y1,
+                                                                  const float* __restrict__ y2, const float* __restrict__ gate, int64_t ld_gate,
+                                                                  const float* __restrict__ rows, int64_t ld_rows, const float* __restrict__ weights,
+                                                                  const int32_t* __restrict__ row_of, int top, const T* __restrict__ pass,
+                                                                  const T* __restrict__ norm_a, const T* __restrict__ norm_b, T* __restrict__ typed_a,
+                                                                  T* __restrict__ typed_b, int W, float eps) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) float row[];
+  __shared__ float red[32];
+  const int64_t t = blockIdx.x;
+  const float s2 = y2 ? (gate ? sigmoid_f(gate[t * ld_gate]) : 1.f) : 0.f;
+  // the identity picks share one weight: their row is read once
+  float w_pass = 0.f, w_k[kPicks];
+  const float* src[kPicks];
+#pragma unroll
+  for (int k = 0; k < kPicks; ++k) {
+    src[k] = nullptr;
+    w_k[k] = 0.f;
+    if (k < top) {
+      const int r = row_of[t * top + k];
+      const float w = weights[t * top + k];
+      if (r >= 0) { src[k] = rows + (int64_t)r * ld_rows; w_k[k] = w; }
+      else w_pass += w;
+    }
+  }
+  float q = 0.f;
+  for (int i = threadIdx.x * VEC; i < W; i += kRowThreads * VEC) {
+    float r[VEC], v[VEC];
+    ld_vec<VEC>((init ? init : x) + t * W + i, r);
+    if (y1) {
+      ld_vec<VEC>(y1 + t * W + i, v);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) r[k] += v[k];
+    }
+    if (y2) {
+      ld_vec<VEC>(y2 + t * W + i, v);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) r[k] = fmaf(s2, v[k], r[k]);
+    }
+    if (w_pass != 0.f) {
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) r[k] = fmaf(w_pass, ldf(pass + t * W + i + k), r[k]);
+    }
+#pragma unroll
+    for (int e = 0; e < kPicks; ++e) {
+      if (e >= top) break;
+      if (src[e] == nullptr) continue;
+      ld_vec<VEC>(src[e] + i, v);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) r[k] = fmaf(w_k[e], v[k], r[k]);
+    }
+    st_vec<float, VEC>(x + t * W + i, r);
+    if (norm_a || norm_b) {
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) q += r[k] * r[k];
+      st_vec<float, VEC>(row + i, r);
+    }
+  }
+  if (!norm_a && !norm_b) return;
+  const float rstd = 1.f / sqrtf(block_sum(q, red) / W + eps);
+  for (int i = threadIdx.x * VEC; i < W; i += kRowThreads * VEC) {   // every thread reads back what it wrote itself
+    float r[VEC], v[VEC];
+    ld_vec<VEC>(row + i, r);
+    if (norm_a) {
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) v[k] = r[k] * rstd * ldf(norm_a + i + k);
+      st_vec<T, VEC>(typed_a + t * W + i, v);
+    }
+    if (norm_b) {
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) v[k] = r[k] * rstd * ldf(norm_b + i + k);
+      st_vec<T, VEC>(typed_b + t * W + i, v);
+    }
+  }
+}
+
+// z <- cap * tanh(z / cap) in place (logits)
+__global__ void __launch_bounds__(256) soft_cap_kernel(float* __restrict__ z, int64_t n, float cap) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t stride = (int64_t)gridDim.x * 256;
+  for (int64_t i = (int64_t)blockIdx.x * 256 + threadIdx.x; i < n; i += stride) z[i] = cap * tanhf(z[i] / cap);
+}
+
 // out = act(in) element by element over rows of F columns (in may be a column slice: leading dimension ld_in);
 // act 0: SiLU, 1: GELU (tanh form), 2: tanh, 3: relu squared, 4: none (a copy or a change of type).  Evaluated in fp32.
 template <int ACT>
@@ -782,6 +876,47 @@ extern "C" int b200_seq_branches_step(float* x, const float* init, const float* 
   else if (dt == B200_DT_BF16) { if (vec) BST(__nv_bfloat16, 4); else BST(__nv_bfloat16, 1); }
   else { b200_set_last_error("unknown element type"); return B200_ERR_ARG; }
 #undef BST
+  b200_count_launches(1);
+  return B200_OK;
+}
+
+// x fp32 [T, W] in place, or from `init`; y1, y2 fp32 [T, W]; gate: one fp32 logit per token (stride ld_gate); rows fp32 (leading dimension
+// ld_rows), weights fp32 [T, top], row_of int32 [T, top] (-1: the pick adds `pass`, [T, W] of type dt), top <= 16; norm_a / norm_b [W] with
+// typed_a / typed_b [T, W] of type dt; every pointer but x may be NULL.
+extern "C" int b200_seq_halves_step(float* x, const float* init, const float* y1, const float* y2, const float* gate, int64_t ld_gate, const float* rows,
+                                    int64_t ld_rows, const float* weights, const int32_t* row_of, int top, const void* pass, const void* norm_a,
+                                    const void* norm_b, int dt, void* typed_a, void* typed_b, int64_t T, int64_t W, float eps, void* stream) {
+  if (T == 0) return B200_OK;
+  if (!row_of) top = 0;
+  if (W > 40000 || top > kPicks || (norm_a && !typed_a) || (norm_b && !typed_b) || (top > 0 && (!rows || !weights || !pass))) {
+    b200_set_last_error("seq_halves_step: width <= 40000, at most 16 picks, a norm needs its row, picks need rows, weights and the router's input");
+    return B200_ERR_ARG;
+  }
+  const size_t smem = (size_t)((W + 3) & ~3) * 4;
+#define HST(E, V)                                                                                                                       \
+  do {                                                                                                                                  \
+    static bool cfg = false;                                                                                                            \
+    if (!cfg) { cudaFuncSetAttribute(halves_step_kernel<E, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024); cfg = true; }  \
+    B200_LAUNCH((halves_step_kernel<E, V>), dim3((unsigned)T), dim3(kRowThreads), smem, (cudaStream_t)stream, x, init, y1, y2, gate, ld_gate, rows, \
+                ld_rows, weights, row_of, top, (const E*)pass, (const E*)norm_a, (const E*)norm_b, (E*)typed_a, (E*)typed_b, (int)W, eps); \
+  } while (0)
+  const bool vec = W % 4 == 0 && ld_rows % 4 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(init) | reinterpret_cast<uintptr_t>(y1) | reinterpret_cast<uintptr_t>(y2) |
+                     reinterpret_cast<uintptr_t>(rows) | reinterpret_cast<uintptr_t>(typed_a) | reinterpret_cast<uintptr_t>(typed_b)) & 15) == 0;
+  if (dt == B200_DT_F32) { if (vec) HST(float, 4); else HST(float, 1); }
+  else if (dt == B200_DT_BF16) { if (vec) HST(__nv_bfloat16, 4); else HST(__nv_bfloat16, 1); }
+  else { b200_set_last_error("unknown element type"); return B200_ERR_ARG; }
+#undef HST
+  b200_count_launches(1);
+  return B200_OK;
+}
+
+// z fp32, n values in place: cap * tanh(z / cap)
+extern "C" int b200_seq_soft_cap(float* z, int64_t n, float cap, void* stream) {
+  if (n == 0) return B200_OK;
+  if (!(cap > 0.f)) { b200_set_last_error("seq_soft_cap: the cap must be positive"); return B200_ERR_ARG; }
+  const int64_t blocks = (n + 1023) / 1024;
+  B200_LAUNCH(soft_cap_kernel, dim3((unsigned)(blocks < 148 * 8 ? blocks : 148 * 8)), dim3(256), 0, (cudaStream_t)stream, z, n, cap);
   b200_count_launches(1);
   return B200_OK;
 }

@@ -9,7 +9,7 @@
 //
 //   qk_rot_prepare_kernel : from a token's projected row [q | k | v] (fp32): RMS norm over the WHOLE q projection and over the
 //                           whole k projection (one statistic for all heads, a weight per column), rotation of the first
-//                           `rot` columns of every head in the rotate-half layout (column i pairs with column i + rot/2; the
+//                           `rot` columns of every head (column i pairs with column i + rot/2, or with its neighbour; the
 //                           cos / sin tables carry frequency scaling and amplitude), keys and values into the token's cache
 //                           slot, queries into a dense fp32 buffer.  Optionally the values turn as well, by their own position
 //                           over the first `v_rot` columns of every value head (halves or neighbouring columns as pairs).
@@ -32,7 +32,7 @@ __global__ void __launch_bounds__(kTalkPrepThreads) qk_rot_prepare_kernel(
     const float* __restrict__ src, int64_t ld, int col_q, int col_k, int col_v, int H, int G, int d, int dv, const T* __restrict__ qnorm_w,
     const T* __restrict__ knorm_w, int whole_norm, float eps, const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot,
     const int64_t* __restrict__ position_ids, const int64_t* __restrict__ slot_mapping, T* __restrict__ cache, int64_t RW, int k_off, int v_off,
-    float* __restrict__ q_out, const float* __restrict__ vcos_t, const float* __restrict__ vsin_t, int v_rot, int v_interleaved) {
+    float* __restrict__ q_out, const float* __restrict__ vcos_t, const float* __restrict__ vsin_t, int v_rot, int v_interleaved, int interleaved) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float red[32];
@@ -61,10 +61,11 @@ __global__ void __launch_bounds__(kTalkPrepThreads) qk_rot_prepare_kernel(
     const float r = is_q ? rq : rk;
     float x = v[c] * r * (w ? ldf(w + c) : 1.f);
     if (i < rot) {
-      const int partner = i < half ? c + half : c - half;
+      const bool first = interleaved ? (i & 1) == 0 : i < half;
+      const int apart = interleaved ? 1 : half, partner = first ? c + apart : c - apart;
       const float y = v[partner] * r * (w ? ldf(w + partner) : 1.f);
-      const int f = i < half ? i : i - half;
-      x = i < half ? x * cs[f] - y * sn[f] : x * cs[f] + y * sn[f];
+      const int f = interleaved ? i >> 1 : first ? i : i - half;
+      x = first ? x * cs[f] - y * sn[f] : x * cs[f] + y * sn[f];
     }
     if (is_q) q_out[t * nq + c] = x;
     else if (crow) stf(crow + k_off + c, x);
@@ -623,13 +624,14 @@ __global__ void __launch_bounds__(256) talk_attn_merge_kernel(const float* __res
 using namespace b200::seq;
 
 // src fp32 [T, ld] holds the projections at columns col_q (H * d), col_k (G * d), col_v (G * dv).  whole_norm: RMS norm over each of
-// the q and k projections as a whole (weights per column, may be NULL).  cos / sin fp32 [positions, rot / 2]; rot 0: no rotation.
+// the q and k projections as a whole (weights per column, may be NULL).  cos / sin fp32 [positions, rot / 2]; rot 0: no rotation;
+// interleaved: the pairs of q and k are neighbours, otherwise the rotated columns' two halves.
 // vcos / vsin fp32 [positions, v_rot / 2]: the values' own turn (v_rot 0: stored as projected; v_interleaved: pairs are neighbours).
 extern "C" int b200_seq_qk_rot_prepare(const float* src, int64_t ld, int col_q, int col_k, int col_v, int H, int G, int d, int dv,
                                        const void* qnorm_w, const void* knorm_w, int whole_norm, float eps, const float* cos_t, const float* sin_t,
                                        int rot, const int64_t* position_ids, const int64_t* slot_mapping, void* cache, int dt, int64_t row_width,
                                        int k_off, int v_off, float* q_out, int64_t T, const float* vcos_t, const float* vsin_t, int v_rot,
-                                       int v_interleaved, void* stream) {
+                                       int v_interleaved, int interleaved, void* stream) {
   if (T == 0) return B200_OK;
   if (v_rot < 0 || v_rot > dv || v_rot % 2 != 0 || (v_rot > 0 && (vcos_t == nullptr || vsin_t == nullptr))) {
     b200_set_last_error("seq_qk_rot_prepare: turned value columns must be even, at most the value size, with tables");
@@ -641,7 +643,8 @@ extern "C" int b200_seq_qk_rot_prepare(const float* src, int64_t ld, int col_q, 
   }
   B200_SEQ_DISPATCH(dt, E, B200_LAUNCH((qk_rot_prepare_kernel<E>), dim3((unsigned)T), dim3(kTalkPrepThreads), 0, (cudaStream_t)stream, src, ld, col_q,
                                        col_k, col_v, H, G, d, dv, (const E*)qnorm_w, (const E*)knorm_w, whole_norm, eps, cos_t, sin_t, rot,
-                                       position_ids, slot_mapping, (E*)cache, row_width, k_off, v_off, q_out, vcos_t, vsin_t, v_rot, v_interleaved));
+                                       position_ids, slot_mapping, (E*)cache, row_width, k_off, v_off, q_out, vcos_t, vsin_t, v_rot, v_interleaved,
+                                       interleaved));
   b200_count_launches(1);
   return B200_OK;
 }

@@ -19,9 +19,9 @@ from .utils.dist import initialize_torch_distributed
 from .utils.weights import Weights
 
 FLASH_TYPES = ["llama", "gpt_neox", "gpt_bigcode", "falcon", "RefinedWeb", "RefinedWebModel", "fetotar", "dubesun", "noganex", "nasozen",
-               "nomalorn"]
+               "nomalorn", "tibopel"]
 # families whose config.json is not a transformers configuration: they name themselves with "architecture"
-OWN_CONFIG_ARCHITECTURES = ("Fetotar", "Dubesun", "Noganex", "Nasozen", "Nomalorn")
+OWN_CONFIG_ARCHITECTURES = ("Fetotar", "Dubesun", "Noganex", "Nasozen", "Nomalorn", "Tibopel")
 _TOKENIZER_FILES = ("tokenizer.json", "tokenizer.model", "tokenizer_config.json", "vocab.json")
 
 
@@ -46,6 +46,9 @@ def load_config(model_path: str):
     if raw.get("architecture") == "Nomalorn":
         from .models.custom_modeling.nomalorn_modeling import NomalornConfig
         return NomalornConfig(raw)
+    if raw.get("architecture") == "Tibopel":
+        from .models.custom_modeling.tibopel_modeling import TibopelConfig
+        return TibopelConfig(raw)
     from transformers import AutoConfig
     return AutoConfig.from_pretrained(model_path)
 
@@ -103,7 +106,7 @@ class InferenceEngine:
                 raise NotImplementedError("alibi is not supported by this version of the model")
             from .models.custom_modeling.flash_rw_modeling import FlashRWForCausalLM
             model_class = FlashRWForCausalLM
-        elif model_type in ("fetotar", "dubesun", "noganex", "nasozen", "nomalorn"):
+        elif model_type in ("fetotar", "dubesun", "noganex", "nasozen", "nomalorn", "tibopel"):
             if quantize is not None:
                 raise ValueError(f"{model_type} checkpoints are served in bfloat16 or float32")
             if dtype not in (torch.bfloat16, torch.float32):
@@ -116,8 +119,10 @@ class InferenceEngine:
                 from .models.custom_modeling.noganex_modeling import NoganexForCausalLM as model_class
             elif model_type == "nasozen":
                 from .models.custom_modeling.nasozen_modeling import NasozenForCausalLM as model_class
-            else:
+            elif model_type == "nomalorn":
                 from .models.custom_modeling.nomalorn_modeling import NomalornForCausalLM as model_class
+            else:
+                from .models.custom_modeling.tibopel_modeling import TibopelForCausalLM as model_class
         self._config.quantize = quantize
         self.process_group = initialize_torch_distributed(self.world_size, self.rank)
         self.master = self.rank == 0

@@ -32,6 +32,7 @@ class RaggedDecoderForCausalLM(nn.Module):
     logits_dtype = torch.float32
     scratch = _NoScratch()        # nothing of the fused step is ever re-allocated
     logit_scale = 1.0             # logits = head(final_norm(x)) * logit_scale
+    logit_softcap = 0.0           # > 0: then cap * tanh(logits / cap)
 
     @property
     def fused_greedy_enabled(self) -> bool:
@@ -126,4 +127,6 @@ class RaggedDecoderForCausalLM(nn.Module):
         logits = ops.linear(self.model.final_norm(x), self.head, out_dtype=torch.float32)
         if self.logit_scale != 1.0:
             logits.mul_(self.logit_scale)
+        if self.logit_softcap > 0.0:
+            ops.soft_cap(logits, self.logit_softcap)
         return logits, kv

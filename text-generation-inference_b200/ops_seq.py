@@ -70,10 +70,13 @@ def _gemm_workspace(device, N: int, K: int) -> torch.Tensor:
     return ws
 
 
+ACT_SILU, ACT_GELU_TANH, ACT_TANH, ACT_RELU2, ACT_NONE = 0, 1, 2, 3, 4
+
+
 def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None,
-           out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """x [M, K] @ w [N, K]^T -> [M, N], fp32 accumulation.  bfloat16 operands go to the tcgen05 product (csrc/gemm_f16.cu,
-    output bfloat16 or fp32) when they are dense and K is a multiple of 8 of at least 64; everything else - float32 operands
+           out: Optional[torch.Tensor] = None, act: int = ACT_NONE) -> torch.Tensor:
+    """act(x [M, K] @ w [N, K]^T) -> [M, N], fp32 accumulation (act: ACT_NONE or ACT_RELU2).  bfloat16 operands go to the tcgen05 product
+    (csrc/gemm_f16.cu, output bfloat16 or fp32) when they are dense and K is a multiple of 8 of at least 64; everything else - float32 operands
     (a true 32-bit product), row-strided slices, small or odd K - to the plain product with ascending-k accumulation."""
     _cuda(x, w, bias)
     assert x.dim() == 2 and w.dim() == 2 and x.stride(1) == 1 and w.stride(1) == 1 and x.shape[1] == w.shape[1]
@@ -81,17 +84,18 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
     N = w.shape[0]
     if out is None:
         out = torch.empty(M, N, dtype=out_dtype or x.dtype, device=x.device)
-    assert out.stride(1) == 1
+    assert out.stride(1) == 1 and act in (ACT_NONE, ACT_RELU2)
     if (_TC_GEMM and x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and out.dtype in (torch.bfloat16, torch.float32)
             and K % 8 == 0 and K >= 64 and x.is_contiguous() and w.is_contiguous() and out.is_contiguous()
             and (bias is None or bias.dtype == torch.bfloat16) and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0 and M > 0):
         ws = _gemm_workspace(x.device, N, K)
-        _lib.check_seq(_lib.load_seq().b200_gemm_bf16(_ptr(x), _ptr(w), _ptr(bias), _ptr(out), int(out.dtype == torch.float32), M, N, K,
-                                                      _ptr(ws), _stream()), "gemm_bf16")
-        return out
+        fused = act == ACT_RELU2 and out.dtype == torch.bfloat16
+        _lib.check_seq(_lib.load_seq().b200_gemm_bf16(_ptr(x), _ptr(w), _ptr(bias), _ptr(out), 2 if fused else int(out.dtype == torch.float32),
+                                                      M, N, K, _ptr(ws), _stream()), "gemm_bf16")
+        return out if fused or act == ACT_NONE else ff_act(out, act, out=out)
     _lib.check_seq(_lib.load_seq().b200_seq_linear(_ptr(x), _dt(x), x.stride(0), 0, _ptr(w), _dt(w), w.stride(0), 0, _ptr(bias), _ptr(out),
                                                    _dt(out), out.stride(0), 0, M, N, K, 1, _stream()), "seq_linear")
-    return out
+    return out if act == ACT_NONE else ff_act(out, act, out=out)
 
 
 def linear_per_head(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
@@ -200,11 +204,14 @@ def latent_prepare(down: torch.Tensor, col_c: int, col_kr: int, q: torch.Tensor,
         _stream()), "seq_latent_prepare")
 
 
-def latent_attn(q_abs: torch.Tensor, cache: torch.Tensor, step: RaggedStep, R: int, r: int, window: int, scale: float) -> torch.Tensor:
+def latent_attn(q_abs: torch.Tensor, cache: torch.Tensor, step: RaggedStep, R: int, r: int, window: int, scale: float,
+                sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """q_abs fp32 [T, H, R + r], cache [blocks, page, R + r] -> fp32 [T, H, R]: soft-max attention of every token over the cache
-    rows of its own sequence at positions (p - window, p], in latent space."""
-    _cuda(q_abs, cache)
+    rows of its own sequence at positions (p - window, p], in latent space (window 0: all of
+    them).  sink fp32 [H]: exp(sink[h]) joins head h's soft-max denominator (not scaled) and carries no value."""
+    _cuda(q_abs, cache, sink)
     T, H, D = q_abs.shape
+    assert sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.shape == (H,))
     assert D == R + r and cache.shape[-1] == D and q_abs.is_contiguous() and cache.is_contiguous()
     out = torch.empty(T, H, R, dtype=torch.float32, device=q_abs.device)
     lib = _lib.load_seq()
@@ -213,8 +220,8 @@ def latent_attn(q_abs: torch.Tensor, cache: torch.Tensor, step: RaggedStep, R: i
     partial = torch.empty(need.value, dtype=torch.float32, device=q_abs.device) if nsplit > 1 else None
     _lib.check_seq(lib.b200_seq_latent_attn(
         _ptr(q_abs), _ptr(cache), _dt(cache), _ptr(step.block_table), step.block_table.stride(0), _ptr(step.seq_of_token),
-        _ptr(step.position_ids), _ptr(out), T, H, R, r, int(window), float(scale), cache.shape[1], _ptr(partial), nsplit, _stream()),
-        "seq_latent_attn")
+        _ptr(step.position_ids), _ptr(out), T, H, R, r, int(window), float(scale), cache.shape[1], _ptr(partial), nsplit, _ptr(sink),
+        _stream()), "seq_latent_attn")
     return out
 
 
@@ -357,37 +364,43 @@ class MoeRouting:
     ids: torch.Tensor       # [T, top] int32
     weights: torch.Tensor   # [T, top] fp32
     plan: torch.Tensor      # int32 workspace (b200_seq_moe_plan_ints)
+    identity: int = 0       # how many router outputs, after the experts', are identity outputs (picks without a row)
 
 
 def moe_route(logits: torch.Tensor, top: int, *, sigmoid_scores: bool = False, correction: Optional[torch.Tensor] = None,
-              weight_scale: float = 1.0) -> MoeRouting:
+              weight_scale: float = 1.0, softmax_scores: bool = False, identity: int = 0) -> MoeRouting:
     """logits fp32 [T, E] -> the `top` largest per token (ties: the lower expert), weights = soft-max over the picked logits.
     sigmoid_scores: the picks are the largest sigmoid(logit) + correction[expert]; the weights are the picked sigmoid(logit)
-    divided by their sum and multiplied by weight_scale."""
+    divided by their sum and multiplied by weight_scale.  softmax_scores: the same with the soft-max over all E logits instead of
+    the sigmoid.  The last `identity` outputs are picked and weighed like experts but have no row in the plan (the other E - identity are
+    the experts).  logits may be a column slice."""
     _cuda(logits, correction)
-    assert logits.dtype == torch.float32 and logits.is_contiguous()
-    T, E = logits.shape
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1 and 0 <= identity < logits.shape[1] and not (sigmoid_scores and softmax_scores)
+    T, E_all = logits.shape
+    E = E_all - identity
     lib = _lib.load_seq()
     ids = torch.empty(T, top, dtype=torch.int32, device=logits.device)
     weights = torch.empty(T, top, dtype=torch.float32, device=logits.device)
     plan = torch.empty(int(lib.b200_seq_moe_plan_ints(T, E, top)), dtype=torch.int32, device=logits.device)
-    if sigmoid_scores:
-        assert correction is None or (correction.is_contiguous() and correction.shape == (E,))
-        _lib.check_seq(lib.b200_seq_moe_route_scored(_ptr(logits), T, E, top, 1, _ptr(correction), 1 if correction is None else _dt(correction),
-                                                     float(weight_scale), _ptr(ids), _ptr(weights), _ptr(plan), _stream()), "seq_moe_route")
-    else:
-        _lib.check_seq(lib.b200_seq_moe_route(_ptr(logits), T, E, top, _ptr(ids), _ptr(weights), _ptr(plan), _stream()), "seq_moe_route")
-    return MoeRouting(T, E, top, ids, weights, plan)
+    mode = 1 if sigmoid_scores else 2 if softmax_scores else 0
+    assert correction is None or (correction.is_contiguous() and correction.shape == (E_all,))
+    _lib.check_seq(lib.b200_seq_moe_route_scored(_ptr(logits), logits.stride(0), T, E, E_all, top, mode, _ptr(correction),
+                                                 1 if correction is None else _dt(correction), float(weight_scale), _ptr(ids), _ptr(weights),
+                                                 _ptr(plan), _stream()), "seq_moe_route")
+    return MoeRouting(T, E, top, ids, weights, plan, identity)
 
 
-def moe_linear(a: torch.Tensor, w: torch.Tensor, r: MoeRouting, gather: bool, out_dtype: torch.dtype) -> torch.Tensor:
-    """w [E, N, K]; a [T, K] (gather: the row of each pick's token) or [T * top, K] (compact rows) -> [T * top, N] compact rows."""
+def moe_linear(a: torch.Tensor, w: torch.Tensor, r: MoeRouting, gather: bool, out_dtype: torch.dtype, act: int = ACT_NONE) -> torch.Tensor:
+    """w [E, N, K]; a [T, K] (gather: the row of each pick's token) or [T * top, K] (compact rows) -> [T * top, N] compact rows (as many as
+    there are picks of experts), after act (ACT_NONE or ACT_RELU2)."""
     _cuda(a, w)
     E, N, K = w.shape
     assert w.is_contiguous() and a.stride(1) == 1 and a.shape[1] == K and E == r.experts and a.shape[0] == (r.T if gather else r.T * r.top)
+    assert act in (ACT_NONE, ACT_RELU2)
     out = torch.empty(r.T * r.top, N, dtype=out_dtype, device=a.device)
     _lib.check_seq(_lib.load_seq().b200_seq_moe_linear(_ptr(a), _dt(a), a.stride(0), int(gather), _ptr(w), _dt(w), _ptr(out), _dt(out),
-                                                       out.stride(0), _ptr(r.plan), r.T, E, r.top, N, K, _stream()), "seq_moe_linear")
+                                                       out.stride(0), _ptr(r.plan), r.T, E, r.top, N, K, int(act == ACT_RELU2), _stream()),
+                   "seq_moe_linear")
     return out
 
 
@@ -410,7 +423,7 @@ def moe_combine_add(resid: torch.Tensor, mix: Optional[torch.Tensor], y: Optiona
     """resid (fp32, in place) += mix + sum_k weights[t, k] y[row(t, k)]; either addend may be None."""
     _cuda(resid, mix, y)
     assert resid.dtype == torch.float32 and resid.is_contiguous() and (mix is None or (mix.dtype == torch.float32 and mix.is_contiguous()))
-    assert y is None or (y.dtype == torch.float32 and y.stride(1) == 1 and r is not None)
+    assert y is None or (y.dtype == torch.float32 and y.stride(1) == 1 and r is not None and r.identity == 0)
     T, W = resid.shape
     _lib.check_seq(_lib.load_seq().b200_seq_moe_combine_add(
         _ptr(resid), _ptr(mix), _ptr(y), 0 if y is None else y.stride(0), None if y is None else _ptr(r.weights), None if y is None else _ptr(r.plan),
@@ -440,9 +453,6 @@ def cast_rows(x: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
     out = torch.empty(x.shape, dtype=dtype, device=x.device)
     _lib.check_seq(_lib.load_seq().b200_seq_cast_rows(_ptr(x), _ptr(out), _dt(dtype), x.numel(), _stream()), "seq_cast_rows")
     return out
-
-
-ACT_SILU, ACT_GELU_TANH = 0, 1
 
 
 def ff_gate(gate_up: torch.Tensor, act: int) -> torch.Tensor:
@@ -509,13 +519,14 @@ def delta_rows_scan(rows: torch.Tensor, S: torch.Tensor, step: RaggedStep, H: in
 def qk_rot_prepare(src: torch.Tensor, *, col_q: int, col_k: int, col_v: int, heads: int, kv_heads: int, dim: int, vdim: int,
                    q_norm_w: Optional[torch.Tensor], k_norm_w: Optional[torch.Tensor], whole_norm: bool, eps: float, cos: Optional[torch.Tensor],
                    sin: Optional[torch.Tensor], rot: int, step: RaggedStep, cache: torch.Tensor, k_off: int, v_off: int,
-                   v_cos: Optional[torch.Tensor] = None, v_sin: Optional[torch.Tensor] = None, v_rot: int = 0, v_interleaved: bool = False
-                   ) -> torch.Tensor:
+                   v_cos: Optional[torch.Tensor] = None, v_sin: Optional[torch.Tensor] = None, v_rot: int = 0, v_interleaved: bool = False,
+                   interleaved: bool = False) -> torch.Tensor:
     """src fp32 [T, C] = [q | k | v] projections: RMS norm over the whole q and the whole k projection (whole_norm), rotation of the
     first `rot` columns of every head in the rotate-half layout with the cos / sin tables, keys and values into the token's row of
     `cache` [blocks, page, row] (token-major: keys of all key heads from k_off, values from v_off) -> queries fp32 [T, heads, dim].
     v_rot > 0: the first v_rot columns of every value head turn by the token's position as well, with tables of their own
-    (v_cos / v_sin [positions, v_rot / 2]); pairs are column i with i + v_rot / 2, or neighbours (v_interleaved)."""
+    (v_cos / v_sin [positions, v_rot / 2]); pairs are column i with i + v_rot / 2, or neighbours (v_interleaved).  `interleaved`: the
+    pairs of q and k are neighbours."""
     _cuda(src, cache, q_norm_w, k_norm_w, cos, sin, v_cos, v_sin)
     assert src.dtype == torch.float32 and src.stride(1) == 1 and cache.is_contiguous()
     assert rot == 0 or (cos.dtype == torch.float32 and cos.is_contiguous() and sin.is_contiguous() and cos.shape[1] == rot // 2)
@@ -524,7 +535,7 @@ def qk_rot_prepare(src: torch.Tensor, *, col_q: int, col_k: int, col_v: int, hea
     _lib.check_seq(_lib.load_seq().b200_seq_qk_rot_prepare(
         _ptr(src), src.stride(0), col_q, col_k, col_v, heads, kv_heads, dim, vdim, _ptr(q_norm_w), _ptr(k_norm_w), int(whole_norm), float(eps),
         _ptr(cos), _ptr(sin), int(rot), _ptr(step.position_ids), _ptr(step.slot_mapping), _ptr(cache), _dt(cache), cache.shape[-1], k_off, v_off,
-        _ptr(q), step.T, _ptr(v_cos), _ptr(v_sin), int(v_rot), int(v_interleaved), _stream()), "seq_qk_rot_prepare")
+        _ptr(q), step.T, _ptr(v_cos), _ptr(v_sin), int(v_rot), int(v_interleaved), int(interleaved), _stream()), "seq_qk_rot_prepare")
     return q
 
 
@@ -595,15 +606,52 @@ def branches_step(x: torch.Tensor, *, init: Optional[torch.Tensor] = None, branc
     return typed
 
 
-ACT_TANH, ACT_RELU2, ACT_NONE = 2, 3, 4
+def halves_step(x: torch.Tensor, *, init: Optional[torch.Tensor] = None, y1: Optional[torch.Tensor] = None, y2: Optional[torch.Tensor] = None,
+                gate: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, routing: Optional[MoeRouting] = None,
+                passed: Optional[torch.Tensor] = None, norm_a: Optional[torch.Tensor] = None, norm_b: Optional[torch.Tensor] = None,
+                eps: float = 0.0, dtype: Optional[torch.dtype] = None):
+    """One fp32 stream whose layers read it once and add two halves side by side, x [T, W] in place (or started from `init`, then x is only
+    written), in one launch: x += y1 + sigmoid(gate) * y2 + sum_k weights[t, k] * (the pick's row of `rows`, or `passed`[t] for a pick of
+    an identity output); -> (unit_rms(x) * norm_a, unit_rms(x) * norm_b) in the norms' element type, None where a norm is None.  y1, y2
+    fp32 [T, W]; gate fp32, one logit per token (a column slice is fine; None: y2 as it is); rows fp32 as moe_linear leaves them;
+    `passed` (the router's input) has the norms' element type (`dtype` when there is no norm)."""
+    _cuda(x, init, y1, y2, gate, rows, passed, norm_a, norm_b)
+    assert x.dtype == torch.float32 and x.is_contiguous() and x.dim() == 2 and (routing is None) == (rows is None) == (passed is None)
+    T, W = x.shape
+    for t in (init, y1, y2):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.shape == x.shape)
+    assert gate is None or (gate.dtype == torch.float32 and gate.numel() == T)
+    assert rows is None or (rows.dtype == torch.float32 and rows.stride(1) == 1 and rows.shape[1] == W and routing.T == T)
+    norms = [n for n in (norm_a, norm_b) if n is not None]
+    dt = norms[0].dtype if norms else (passed.dtype if passed is not None else dtype or torch.float32)
+    assert all(n.dtype == dt and n.is_contiguous() and n.shape == (W,) for n in norms)
+    assert passed is None or (passed.dtype == dt and passed.is_contiguous() and passed.shape == x.shape)
+    a, b = (None if n is None else torch.empty(T, W, dtype=dt, device=x.device) for n in (norm_a, norm_b))
+    lib = _lib.load_seq()
+    row_of, top = (None, 0) if routing is None else (lib.b200_seq_moe_row_of(_ptr(routing.plan), T, routing.experts, routing.top), routing.top)
+    _lib.check_seq(lib.b200_seq_halves_step(_ptr(x), _ptr(init), _ptr(y1), _ptr(y2), _ptr(gate), 0 if gate is None else gate.stride(0), _ptr(rows),
+                                            0 if rows is None else rows.stride(0), None if routing is None else _ptr(routing.weights), row_of, top,
+                                            _ptr(passed), _ptr(norm_a), _ptr(norm_b), _dt(dt), _ptr(a), _ptr(b), T, W, float(eps), _stream()),
+                   "seq_halves_step")
+    return a, b
 
 
-def ff_act(x: torch.Tensor, act: int, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+def soft_cap(z: torch.Tensor, cap: float) -> torch.Tensor:
+    """fp32 z <- cap * tanh(z / cap) in place"""
+    _cuda(z)
+    assert z.dtype == torch.float32 and z.is_contiguous()
+    _lib.check_seq(_lib.load_seq().b200_seq_soft_cap(_ptr(z), z.numel(), float(cap), _stream()), "seq_soft_cap")
+    return z
+
+
+def ff_act(x: torch.Tensor, act: int, out_dtype: Optional[torch.dtype] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """act(x) element by element (ACT_SILU, ACT_GELU_TANH, ACT_TANH, ACT_RELU2: relu(x)^2, ACT_NONE: x itself), evaluated in fp32; x [T, F]
-    may be a column slice; fp32 rows may come out in another element type."""
+    may be a column slice; fp32 rows may come out in another element type.  `out`: dense rows to write, x itself if that is dense."""
     _cuda(x)
     assert x.dim() == 2 and x.stride(1) == 1
-    out = torch.empty(x.shape, dtype=out_dtype or x.dtype, device=x.device)
+    if out is None:
+        out = torch.empty(x.shape, dtype=out_dtype or x.dtype, device=x.device)
+    assert out.is_contiguous() and out.shape == x.shape
     _lib.check_seq(_lib.load_seq().b200_seq_ff_act(_ptr(x), _dt(x), x.stride(0), _ptr(out), _dt(out), x.shape[0], x.shape[1], int(act), _stream()),
                    "seq_ff_act")
     return out

@@ -34,7 +34,9 @@ def _need_single_rank(weights, what: str):
 class ScaledRotaryTables:
     """cos / sin of position * frequency of every rotated pair, fp32 [positions, dims / 2], grown on demand (which columns form
     pair i - neighbours or halves - is the kernel's business).
-    frequency_i = base^(-2i/dims).  With `scaling` = {factor, original, fast, slow} (YaRN): pairs that turn more than `fast`
+    frequency_i = base^(-2i/dims).  With `scaling` = {factor, original, low, high} (by wavelength, as Llama 3.1 does): a pair whose
+    wavelength is below original / high keeps its frequency, one above original / low is slowed by `factor`, in between the two are
+    blended linearly in original / wavelength.  With `scaling` = {factor, original, fast, slow} (YaRN): pairs that turn more than `fast`
     times over `original` positions keep their frequency, pairs that turn fewer than `slow` times are slowed by `factor`, a
     linear ramp over the pair index in between; cos and sin are multiplied by 0.1 ln(factor) + 1."""
 
@@ -48,7 +50,12 @@ class ScaledRotaryTables:
         i = torch.arange(self.dims // 2, dtype=torch.float64)
         freq = self.base ** (-2.0 * i / self.dims)
         sc = self.scaling
-        if sc:
+        if sc and "low" in sc:
+            turns = float(sc["original"]) * freq / (2.0 * math.pi)      # original / wavelength
+            low, high = float(sc["low"]), float(sc["high"])
+            keep = ((turns - low) / (high - low)).clamp(0.0, 1.0) if high != low else (turns > low).to(freq.dtype)
+            freq = freq / float(sc["factor"]) * (1.0 - keep) + freq * keep
+        elif sc:
             def pair_turning(turns: float) -> float:  # (fractional) pair index that makes `turns` turns over the original length
                 return self.dims * math.log(float(sc["original"]) / (2.0 * math.pi * turns)) / (2.0 * math.log(self.base))
             lo = max(math.floor(pair_turning(float(sc["fast"]))), 0)
@@ -58,7 +65,7 @@ class ScaledRotaryTables:
         return freq
 
     def amplitude(self) -> float:
-        return 0.1 * math.log(float(self.scaling["factor"])) + 1.0 if self.scaling else 1.0
+        return 0.1 * math.log(float(self.scaling["factor"])) + 1.0 if self.scaling and "low" not in self.scaling else 1.0
 
     def tables(self, n_pos: int, device):
         if self._cos is None or self._cos.shape[0] < n_pos or self._cos.device != torch.device(device):
@@ -75,10 +82,13 @@ class LatentAttention(nn.Module):
     key part (`rot_dim`) shared by all heads; queries go through a latent of rank `q_rank`.  Only the normalised latent and the
     rotated key part are cached: `kv_rank + rot_dim` elements per token and layer.  The kernels work in the absorbed form (the
     key up-projection is applied to the query, the value up-projection to the attention output), for prompts and decoding alike.
-    Tensors under `prefix`: dq, dq.norm, uq, dkv, dkv.norm, uk, uv, g (sigmoid gate on the concatenated heads), o."""
+    `window` None: every earlier token is visible.  `gate`: a sigmoid gate on the concatenated heads; `sink`: a logit per head in the
+    soft-max denominator.  `out_dtype`: element type of the result (None: the projections' type).
+    Tensors under `prefix`: dq, dq.norm, uq, dkv, dkv.norm, uk, uv, [g,] [sink,] o."""
 
     def __init__(self, prefix: str, weights, *, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, q_rank: int, scale: float,
-                 window: Optional[int], rotary: ScaledRotaryTables, eps: float):
+                 window: Optional[int], rotary: ScaledRotaryTables, eps: float, gate: bool = True, sink: bool = False,
+                 out_dtype: Optional[torch.dtype] = None):
         super().__init__()
         _need_single_rank(weights, "LatentAttention")
         self.H, self.d, self.r, self.dv, self.R, self.Q = heads, dim, rot_dim, vdim, kv_rank, q_rank
@@ -86,13 +96,18 @@ class LatentAttention(nn.Module):
         if rotary.dims > rot_dim:
             raise ValueError("rotary dims exceed the rotated part")
         get = lambda n: weights.get_tensor(f"{prefix}.{n}")  # noqa: E731
-        self.w_in = torch.cat([get("dq"), get("dkv"), get("g")], 0).contiguous()          # -> [q latent | kv latent | key part | gate]
+        self.gate, self.out_dtype = bool(gate), out_dtype
+        self.w_in = torch.cat([get(n) for n in (("dq", "dkv", "g") if gate else ("dq", "dkv"))], 0).contiguous()   # -> [q latent | kv latent | key part | gate]
         self.dq_norm, self.dkv_norm = get("dq.norm"), get("dkv.norm")
         self.w_uq = get("uq").contiguous()                                               # rows head by head: [dim plain | rot_dim rotated]
         self.w_uk_t = get("uk").view(heads, dim, kv_rank).transpose(1, 2).contiguous()   # [H, R, d]: q~ = Wuk_h^T q_plain
         self.w_uv = get("uv").view(heads, vdim, kv_rank).contiguous()
         self.w_o = get("o").contiguous()
         self.dtype = self.w_o.dtype
+        self.sink = get("sink").float().contiguous() if sink else None
+        if self.w_in.shape[0] != q_rank + kv_rank + rot_dim + (heads * vdim if gate else 0) or self.w_uq.shape != (heads * (dim + rot_dim), q_rank) or \
+                self.w_o.shape[1] != heads * vdim or (sink and self.sink.shape != (heads,)):
+            raise ValueError(f"{prefix}: tensor shapes do not match the head sizes and ranks")
 
     def cache_spec(self) -> LayerCacheSpec:
         return LayerCacheSpec(kind="paged", row_width=self.R + self.r)
@@ -107,12 +122,14 @@ class LatentAttention(nn.Module):
         cos, sin = self.rotary.tables(max_s, h.device)
         ops.latent_prepare(down, Q, Q + R, q, d + r, d, self.dkv_norm, cos, sin, step, store, q_abs, H, R, r, self.rotary.dims, self.eps)
         ops.linear_per_head(q.view(T, H, d + r)[:, :, :d], self.w_uk_t, q_abs[:, :, :R])
-        o_lat = ops.latent_attn(q_abs, store, step, R, r, self.window, self.scale)
+        o_lat = ops.latent_attn(q_abs, store, step, R, r, self.window, self.scale, self.sink)
         o = torch.empty(T, H, dv, dtype=torch.float32, device=h.device)
         ops.linear_per_head(o_lat, self.w_uv, o)
-        gated = ops.group_rmsnorm_gate(o.view(T, H * dv), None, 0, self.eps, self.dtype, gate=down[:, Q + R + r:],
-                                       gate_kind=ops.GATE_SIGMOID_AFTER)
-        return ops.linear(gated, self.w_o)
+        if self.gate:
+            o = ops.group_rmsnorm_gate(o.view(T, H * dv), None, 0, self.eps, self.dtype, gate=down[:, Q + R + r:], gate_kind=ops.GATE_SIGMOID_AFTER)
+        else:
+            o = ops.cast_rows(o.view(T, H * dv), self.dtype)
+        return ops.linear(o, self.w_o, out_dtype=self.out_dtype)
 
 
 class Mamba2Mixer(nn.Module):
@@ -305,33 +322,55 @@ class BucketBiasAttention(nn.Module):
 class RoutedExperts(nn.Module):
     """Mixture of gated experts without biases: router logits in fp32, `top` experts per token.  Routing rule: the largest logits
     with weights = soft-max over the picked logits, or (`sigmoid_scores`) the largest sigmoid(logit) + correction with weights =
-    picked sigmoid(logit) / their sum * `weight_scale`.  Expert: down(act(gate x) . up x), act = the clamped form of
-    `ClampedGatedMLP` (`limit` given: g' sigmoid(alpha g') (u' + 1)) or plain SiLU(g) u (`limit` None).  `forward` returns the
-    experts' outputs as compact rows (expert by expert) with the routing; `ops.moe_combine_add` sums them into the stream.
-    Tensors under `prefix`: router, [correction,] e<j>.gate, e<j>.up, e<j>.down."""
+    picked sigmoid(logit) / their sum * `weight_scale`, or (`softmax_scores`) the same with the soft-max over all router outputs.  The
+    last `identity` router outputs have no tensors: their result is the input.  Expert: down(act(gate x) . up x), act = the clamped form of
+    `ClampedGatedMLP` (`limit` given: g' sigmoid(alpha g') (u' + 1)) or plain SiLU(g) u (`limit` None); or without a gate
+    (`plain` "relu2"): down(relu(up x)^2).  `forward` returns the experts' outputs as compact rows (expert by expert) with the routing;
+    `ops.moe_combine_add` (or `ops.halves_step`, which knows identity outputs) sums them into the stream.  `more_rows`: rows of other
+    products of the same input that run with the router's; `route` returns their fp32 results after the routing.
+    Tensors under `prefix`: router, [correction,] [e<j>.gate,] e<j>.up, e<j>.down."""
 
     dense_rows_per_expert = 64   # average rows per expert from which a step runs one dense product per expert
 
     def __init__(self, prefix: str, weights, *, experts: int, top: int, limit: Optional[float], alpha: float = 1.702,
-                 sigmoid_scores: bool = False, correction: bool = False, weight_scale: float = 1.0):
+                 sigmoid_scores: bool = False, correction: bool = False, weight_scale: float = 1.0, softmax_scores: bool = False,
+                 identity: int = 0, plain: Optional[str] = None, more_rows: Optional[torch.Tensor] = None):
         super().__init__()
         _need_single_rank(weights, "RoutedExperts")
+        if plain not in (None, "relu2"):
+            raise NotImplementedError(f"expert activation {plain!r}")
+        self.softmax_scores, self.identity, self.plain = bool(softmax_scores), int(identity), plain
         self.E, self.top, self.limit, self.alpha = int(experts), int(top), None if limit is None else float(limit), float(alpha)
         self.sigmoid_scores, self.weight_scale = bool(sigmoid_scores), float(weight_scale)
         get = lambda n: weights.get_tensor(f"{prefix}.{n}")  # noqa: E731
         self.correction = get("correction").contiguous() if correction else None
         self.w_router = get("router").contiguous()
-        self.w_gate_up = torch.stack([torch.cat([get(f"e{e}.gate"), get(f"e{e}.up")], 0) for e in range(self.E)]).contiguous()
+        # the first product of every expert: [gate; up], or up alone
+        self.w_gate_up = torch.stack([get(f"e{e}.up") if plain else torch.cat([get(f"e{e}.gate"), get(f"e{e}.up")], 0) for e in range(self.E)]).contiguous()
         self.w_down = torch.stack([get(f"e{e}.down") for e in range(self.E)]).contiguous()
-        if self.w_router.shape[0] != self.E:
-            raise ValueError(f"{prefix}.router: one row per expert expected")
+        self.n_route = self.E + self.identity
+        if self.w_router.shape[0] != self.n_route or (correction and self.correction.shape != (self.n_route,)):
+            raise ValueError(f"{prefix}.router: one row per expert and identity output expected")
+        if more_rows is not None:
+            self.w_router = torch.cat([self.w_router, more_rows], 0).contiguous()
 
     def _act(self, gu: torch.Tensor) -> torch.Tensor:
+        if self.plain:
+            return gu      # the first product applies it
         return ops.ff_gate(gu, ops.ACT_SILU) if self.limit is None else ops.ff_clamped_gate(gu, self.limit, self.alpha)
 
+    def route(self, h: torch.Tensor):
+        """-> the step's routing, and fp32 [T, n] of `more_rows`"""
+        z = ops.linear(h, self.w_router, out_dtype=torch.float32)
+        return ops.moe_route(z[:, :self.n_route], self.top, sigmoid_scores=self.sigmoid_scores, correction=self.correction,
+                             weight_scale=self.weight_scale, softmax_scores=self.softmax_scores, identity=self.identity), z[:, self.n_route:]
+
     def forward(self, h: torch.Tensor):
-        routing = ops.moe_route(ops.linear(h, self.w_router, out_dtype=torch.float32), self.top, sigmoid_scores=self.sigmoid_scores,
-                                correction=self.correction, weight_scale=self.weight_scale)
+        routing, _ = self.route(h)
+        return self.experts(h, routing), routing
+
+    def experts(self, h: torch.Tensor, routing) -> torch.Tensor:
+        act1 = ops.ACT_RELU2 if self.plain else ops.ACT_NONE
         rows = h.shape[0] * self.top
         if h.dtype == torch.bfloat16 and rows >= self.dense_rows_per_expert * self.E and not torch.cuda.is_current_stream_capturing():
             # prompts: enough rows per expert for the tcgen05 product (ops.linear) to pay - one product per expert over its run of
@@ -341,15 +380,36 @@ class RoutedExperts(nn.Module):
             gu = torch.empty(rows, self.w_gate_up.shape[1], dtype=h.dtype, device=h.device)
             for e in range(self.E):
                 if offs[e + 1] > offs[e]:
-                    ops.linear(a[offs[e]:offs[e + 1]], self.w_gate_up[e], out=gu[offs[e]:offs[e + 1]])
+                    ops.linear(a[offs[e]:offs[e + 1]], self.w_gate_up[e], out=gu[offs[e]:offs[e + 1]], act=act1)
             act = self._act(gu)
             y = torch.empty(rows, self.w_down.shape[1], dtype=torch.float32, device=h.device)
             for e in range(self.E):
                 if offs[e + 1] > offs[e]:
                     ops.linear(act[offs[e]:offs[e + 1]], self.w_down[e], out=y[offs[e]:offs[e + 1]])
-            return y, routing
-        gu = ops.moe_linear(h, self.w_gate_up, routing, gather=True, out_dtype=h.dtype)
-        return ops.moe_linear(self._act(gu), self.w_down, routing, gather=False, out_dtype=torch.float32), routing
+            return y
+        gu = ops.moe_linear(h, self.w_gate_up, routing, gather=True, out_dtype=h.dtype, act=act1)
+        return ops.moe_linear(self._act(gu), self.w_down, routing, gather=False, out_dtype=torch.float32)
+
+
+class RoutedSharedFeedForward(nn.Module):
+    """Squared-ReLU experts by corrected soft-max scores, some router outputs being the identity, beside an expert that every token uses
+    times sigmoid(W_sg h), one number per token.  `forward` returns what `ops.halves_step` adds to the stream: the shared expert's result
+    (y2) with its gate logits, the routed experts' rows with the routing, and the input that identity picks pass on.
+    Tensors under `prefix`: router, correction, e<j>.up, e<j>.down [, shared.up, shared.down, shared.sg]."""
+
+    def __init__(self, prefix: str, weights, *, experts: int, identity: int, top: int, shared: bool):
+        super().__init__()
+        gate_row = weights.get_tensor(f"{prefix}.shared.sg") if shared else None
+        self.routed = RoutedExperts(prefix, weights, experts=experts, top=top, limit=None, softmax_scores=True, correction=True, identity=identity,
+                                    plain="relu2", more_rows=gate_row)
+        self.shared = PlainMLP(f"{prefix}.shared", weights, activation="relu2") if shared else None
+
+    def forward(self, h: torch.Tensor) -> dict:
+        routing, more = self.routed.route(h)
+        out = {"rows": self.routed.experts(h, routing), "routing": routing, "passed": h}
+        if self.shared is not None:
+            out.update(y2=self.shared(h), gate=more[:, 0])
+        return out
 
 
 class GatedMLP(nn.Module):
@@ -467,27 +527,28 @@ class SinkRotaryAttention(nn.Module):
     with column i + dims / 2).  Cached per token: rotated keys and turned values of all key heads (token-major row); per
     sequence: the last conv - 1 projected rows (fp32).
     Every part but the soft-max is optional: `sink`, `head_gate`, `qk_norm` False and `rotary` / `value_rotary` None leave theirs out,
-    `bias` adds q.b / k.b / v.b to the projections, `window` (the last so many keys) and `chunk` (keys of the query's own chunk of so
+    `bias` adds q.b / k.b / v.b to the projections, `out_bias` o.b to the output product of `forward`, `qk_pairs` says how q and k rotate
+    ("halves", or "interleaved": neighbouring columns), `window` (the last so many keys) and `chunk` (keys of the query's own chunk of so
     many positions, counted from position 0) are the masks.
     A mixer that can share its input and output products with a neighbour: `in_rows()` are the rows it adds to the input
     projection (`in_bias()` their biases), `from_projection` continues from the fp32 projection and leaves the gated heads, times
     `out_scale`, in `out`; `w_o` finishes.
-    Tensors under `prefix`: q, k, v, [q.b, k.b, v.b,] [q.conv, k.conv, v.conv,] [q.norm, k.norm,] [sink,] [g,] o."""
+    Tensors under `prefix`: q, k, v, [q.b, k.b, v.b,] [q.conv, k.conv, v.conv,] [q.norm, k.norm,] [sink,] [g,] o [, o.b]."""
 
     def __init__(self, prefix: str, weights, *, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, rotary: Optional[ScaledRotaryTables],
                  value_rotary: Optional[ScaledRotaryTables], value_pairs: str = "halves", conv: int = 0, window: Optional[int] = None,
                  sink: bool = True, head_gate: bool = True, eps: float = 1e-6, qk_norm: bool = True, bias: bool = False,
-                 chunk: Optional[int] = None):
+                 chunk: Optional[int] = None, out_bias: bool = False, qk_pairs: str = "halves"):
         super().__init__()
         _need_single_rank(weights, "SinkRotaryAttention")
         if heads % kv_heads:
             raise ValueError("heads must be a multiple of kv_heads")
-        if value_pairs not in ("halves", "interleaved"):
-            raise ValueError("value_pairs is 'halves' or 'interleaved'")
+        if value_pairs not in ("halves", "interleaved") or qk_pairs not in ("halves", "interleaved"):
+            raise ValueError("value_pairs and qk_pairs are 'halves' or 'interleaved'")
         self.H, self.G, self.d, self.dv, self.taps = int(heads), int(kv_heads), int(dim), int(vdim), int(conv or 0)
         self.scale, self.rotary, self.value_rotary, self.window, self.eps = float(scale), rotary, value_rotary, int(window or 0), float(eps)
         self.chunk = int(chunk or 0)
-        self.value_interleaved = value_pairs == "interleaved"
+        self.value_interleaved, self.qk_interleaved = value_pairs == "interleaved", qk_pairs == "interleaved"
         if rotary is not None and rotary.dims > dim:
             raise ValueError("rotary dims exceed the head size")
         if value_rotary is not None and value_rotary.dims > vdim:
@@ -508,6 +569,7 @@ class SinkRotaryAttention(nn.Module):
         self.sink = get("sink").float().contiguous() if sink else None
         self.w_o = get("o").contiguous()
         self.dtype = self.w_o.dtype
+        self.b_o = get("o.b").contiguous() if out_bias else None
         self.n_out = self.H * self.dv
         if self.w_in.shape[0] != self.n_in or (self.conv_w is not None and self.conv_w.shape != (self.channels, self.taps)) or \
                 self.w_o.shape[1] != self.n_out or (self.sink is not None and self.sink.shape != (self.H,)) or \
@@ -541,7 +603,8 @@ class SinkRotaryAttention(nn.Module):
         q = ops.qk_rot_prepare(c, col_q=cq, col_k=cq + self.cq, col_v=cq + self.cq + self.ck, heads=self.H, kv_heads=self.G, dim=self.d,
                                vdim=self.dv, q_norm_w=self.q_norm, k_norm_w=self.k_norm, whole_norm=self.qk_norm, eps=self.eps, cos=cos, sin=sin,
                                rot=self.rotary.dims if self.rotary is not None else 0, step=step, cache=pages, k_off=0, v_off=self.ck,
-                               v_cos=vcos, v_sin=vsin, v_rot=vr.dims if vr is not None else 0, v_interleaved=self.value_interleaved)
+                               v_cos=vcos, v_sin=vsin, v_rot=vr.dims if vr is not None else 0, v_interleaved=self.value_interleaved,
+                               interleaved=self.qk_interleaved)
         a = ops.talk_attn(q, pages, step, kv_heads=self.G, vdim=self.dv, k_off=0, v_off=self.ck, scale=self.scale, chunk=self.chunk,
                           window=self.window, sink=self.sink)
         gate = u[:, col0 + self.channels:col0 + self.channels + self.H] if self.head_gate else None
@@ -553,7 +616,7 @@ class SinkRotaryAttention(nn.Module):
         u = ops.linear(h, self.w_in, self.b_in, out_dtype=torch.float32)
         o = torch.empty(step.T, self.n_out, dtype=self.dtype, device=h.device)
         self.from_projection(u, 0, step, pages, state, max_s, o)
-        return ops.linear(o, self.w_o, out_dtype=torch.float32)
+        return ops.linear(o, self.w_o, self.b_o, out_dtype=torch.float32)
 
 
 class MinGRUMixer(nn.Module):
@@ -802,4 +865,8 @@ class PlainMLP(nn.Module):
         self.b_up, self.b_down = (weights.get_tensor(f"{prefix}.{n}.b").contiguous() if bias else None for n in ("up", "down"))
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
-        return ops.linear(ops.ff_act(ops.linear(h, self.w_up, self.b_up), self.act), self.w_down, self.b_down, out_dtype=torch.float32)
+        if self.act == ops.ACT_RELU2:      # inside the product's epilogue where that is possible
+            up = ops.linear(h, self.w_up, self.b_up, act=self.act)
+        else:
+            up = ops.ff_act(ops.linear(h, self.w_up, self.b_up), self.act)
+        return ops.linear(up, self.w_down, self.b_down, out_dtype=torch.float32)
