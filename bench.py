@@ -1098,12 +1098,16 @@ def _stream_family_measure(raw, cfg, op_names, PB, PL, DB, DL, K, Wm, timed, lib
     for _ in range(Wm):
         prefill_once()
     pre_ms = timed(prefill_once, K)
-    log = []
+    log, routes = [], []
+    route = ops_seq.moe_route
+    ops_seq.moe_route = lambda *a, **k: (routes.append(route(*a, **k)), routes[-1])[1]
     saved = _timed_ops(ops_seq, op_names, log)
     prefill_once()
     pre_ops = _by_op(log)
     for n, fn in saved.items():
         setattr(ops_seq, n, fn)
+    ops_seq.moe_route = route
+    pre_rows = sum(int((r.ids < r.experts).sum()) for r in routes)    # picks of experts (the rest are identity outputs), all layers
     sids, _ = model.step_ragged([None] * DB, prompt(DB, DL), [])
     nxt = [[t[0]] for t in prompt(DB, 1)]
 
@@ -1121,7 +1125,7 @@ def _stream_family_measure(raw, cfg, op_names, PB, PL, DB, DL, K, Wm, timed, lib
     for n, fn in saved.items():
         setattr(ops_seq, n, fn)
     ops_seq.moe_route = route
-    picked = sum(len(set(r.ids.flatten().tolist())) for r in routes)
+    picked = sum(len({e for e in r.ids.flatten().tolist() if e < r.experts}) for r in routes)
     model.kv_cache_manager.free_sequences(sids)
     with torch.inference_mode():   # the serving path: from_pb -> generate_token, plain greedy, replayed as one CUDA graph
         gpb = make_batch_pb(DB, DL, Wm + K + 8)
@@ -1138,7 +1142,7 @@ def _stream_family_measure(raw, cfg, op_names, PB, PL, DB, DL, K, Wm, timed, lib
     gc.collect()
     torch.cuda.empty_cache()
     return {"pre_ms": pre_ms, "pre_ops": pre_ops, "dec_ms": dec_ms, "dec_ops": dec_ops, "graph_ms": graph_ms, "dec_k": dec_k, "dec_total": dec_total,
-            "picked": picked}
+            "picked": picked, "pre_rows": pre_rows}
 
 
 def _noganex_side(width, env):
@@ -1400,6 +1404,90 @@ def run_nomalorn_compare(args):
     return env["report"]("nomalorn_compare", results)
 
 
+def _latent_lines(pre_ops, dec_k, m, PB, PL, DB, ctx, n, hbm, tens, us):
+    """the two lines of latent attention: absorbed form, every head reads the same row of the cache (m: mixer sizes, n layers of it)"""
+    D, R, H = m["kv_rank"] + m["rot_dim"], m["kv_rank"], m["heads"]
+    flops = n * PB * (PL * (PL + 1) // 2) * H * (D + R) * 2
+    t, per_head = us(dec_k, "latent_attn"), us(dec_k, "linear_kernel", "group_gemm")
+    ph_flops = n * PB * PL * H * R * (m["dim"] + m["vdim"]) * 2
+    return {"latent_attn prefill": {"ms": pre_ops["latent_attn"], "tflops": flops / pre_ops["latent_attn"] / 1e9,
+                                    "of_measured_tensor": flops / (pre_ops["latent_attn"] * 1e-3) / tens},
+            "latent_attn decode": {"us": t, "of_measured_hbm": n * DB * ctx * D * 2 / (max(t, 1e-9) * 1e-6) / hbm},
+            "linear_per_head prefill": {"ms": pre_ops["linear_per_head"], "tflops": ph_flops / pre_ops["linear_per_head"] / 1e9,
+                                        "of_measured_tensor": ph_flops / (pre_ops["linear_per_head"] * 1e-3) / tens},
+            "linear_per_head decode": {"us": per_head, "of_measured_hbm": n * H * R * (m["dim"] + m["vdim"]) * 2 / (max(per_head, 1e-9) * 1e-6) / hbm}}
+
+
+def _fetotar_latent_side(width, env):
+    """Fetotar's latent-attention layer as the partner of --tibopel-compare (latent attention and its per-head products only)"""
+    from tgis_b200.models.custom_modeling import fetotar_modeling
+    from tgis_b200.utils.synthetic import fetotar_config
+    raw = fetotar_config(f"fetotar-w{width}")
+    names = ["linear", "linear_per_head", "embed_scale", "layernorm", "layernorm_into_residual", "group_rmsnorm_gate", "ff_clamped_gate", "token_side",
+             "latent_prepare", "latent_attn", "causal_conv_silu", "ssm_scan", "mlstm_scan"]
+    PB, PL, DB, DL, K, Wm = (env[k] for k in ("PB", "PL", "DB", "DL", "K", "Wm"))
+    r = _stream_family_measure(raw, fetotar_modeling.FetotarConfig(raw), names, PB, PL, DB, DL, K, Wm, env["timed"], env["lib"])
+    kernels = _latent_lines(r["pre_ops"], r["dec_k"], raw["layers"][1]["mixer"], PB, PL, DB, env["ctx"], 1, env["hbm"], env["tens"], env["us"])
+    return env["common"](f"fetotar-w{width}", raw, r, kernels, {"latent_layers": 1})
+
+
+def run_tibopel_compare(args):
+    """Tibopel (bfloat16) beside the closest families of the engine at equal width and number of layers on random weights: Noganex (chunked
+    attention over token-major rows, routed and shared experts, an fp32 stream) and, for its latent attention, Fetotar.  Prefill of 4 x 1024
+    tokens and decode of 32 sequences at context 1024, measured as --noganex-compare measures its pair, with the achieved FLOP/s or
+    bytes/s of the kernels that carry a step against the measured peaks."""
+    import tgis_b200  # noqa: F401
+    from tgis_b200.models.custom_modeling import tibopel_modeling
+    from tgis_b200.utils.synthetic import tibopel_config
+
+    env = _stream_compare_env(args)
+    PB, PL, DB, DL, K, Wm, ctx = (env[k] for k in ("PB", "PL", "DB", "DL", "K", "Wm", "ctx"))
+    timed, lib, hbm, tens, common, us = (env[k] for k in ("timed", "lib", "hbm", "tens", "common", "us"))
+    results = []
+    for width in env["widths"]:
+        raw = tibopel_config(f"tibopel-w{width}")
+        names = ["linear", "linear_per_head", "embed_scale", "halves_step", "qk_rot_prepare", "talk_attn", "heads_turn_gate", "group_rmsnorm_gate",
+                 "latent_prepare", "latent_attn", "cast_rows", "moe_route", "moe_gather_rows", "moe_linear", "ff_act", "rmsnorm_rows", "soft_cap"]
+        r = _stream_family_measure(raw, tibopel_modeling.TibopelConfig(raw), names, PB, PL, DB, DL, K, Wm, timed, lib)
+        shapes, L = tibopel_modeling.tensor_shapes(raw), raw["layers"]
+        attn = [l["mixer"] for l in L if l["type"] == "attention"]
+        latent = [l["mixer"] for l in L if l["type"] == "latent_attention"]
+        attn_flops = sum(PB * (PL * (PL + 1) // 2) * m["heads"] * (m["dim"] + m["vdim"]) * 2 for m in attn)
+        attn_row = sum(m["kv_heads"] * (m["dim"] + m["vdim"]) for m in attn)       # elements a decoding token reads per cached token
+        moe = L[0]["mlp"]
+        expert_w, T, top = 2 * width * moe["expert"]["ff"], PB * PL, moe["router"]["top"]
+        dense_w = sum(a * b for n, (a, *rest) in shapes.items() for b in rest[:1] if ".mlp.e" not in n and n not in ("embed", "head")
+                      and not n.endswith((".uk", ".uv")))
+        head_w = shapes["head"][0] * shapes["head"][1]
+        pre, dk = r["pre_ops"], r["dec_k"]
+        # the picks that are experts (identity outputs cost nothing): counted in the prefill that was timed
+        rows = r["pre_rows"]
+        lin_flops, moe_flops = 2 * T * dense_w + 2 * PB * head_w, 2 * rows * expert_w
+        if "moe_linear" not in pre:      # one dense product per expert: inside `linear`
+            lin_flops, moe_flops = lin_flops + moe_flops, 0
+        # a layer's boundary: stream in and out, the mixer's and the shared expert's results, the picked rows, the passed row, two typed rows out
+        stream_b = sum(width * (8 + 4 + 4 + 4 * top + 2 + 4) for _ in L)
+        a_us, m_us, g_us, h_us = us(dk, "talk_attn"), us(dk, "moe_linear"), dk.get("gemm_f16_kernel", 0.0), us(dk, "halves_step")
+        kernels = {
+            "talk_attn prefill": {"ms": pre["talk_attn"], "tflops": attn_flops / pre["talk_attn"] / 1e9,
+                                  "of_measured_tensor": attn_flops / (pre["talk_attn"] * 1e-3) / tens},
+            "talk_attn decode": {"us": a_us, "of_measured_hbm": DB * ctx * attn_row * 2 / (max(a_us, 1e-9) * 1e-6) / hbm},
+            **_latent_lines(pre, dk, latent[0], PB, PL, DB, ctx, len(latent), hbm, tens, us),
+            "linear prefill": {"ms": pre["linear"], "of_measured_tensor": lin_flops / (pre["linear"] * 1e-3) / tens},
+            "linear decode (tcgen05 projections)": {"us": g_us, "of_measured_hbm": (dense_w + head_w) * 2 / (max(g_us, 1e-9) * 1e-6) / hbm},
+            "moe_linear decode (grouped, picked experts' weights once)": {"us": m_us, "experts_picked_all_layers": r["picked"], "of_measured_hbm":
+                                                                          r["picked"] * expert_w * 2 / (max(m_us, 1e-9) * 1e-6) / hbm},
+            "halves_step prefill": {"ms": pre["halves_step"], "of_measured_hbm": T * stream_b / (pre["halves_step"] * 1e-3) / hbm},
+            "halves_step decode": {"us": h_us, "launches": len(L) + 1, "of_measured_hbm": DB * stream_b / (max(h_us, 1e-9) * 1e-6) / hbm},
+        }
+        if moe_flops:
+            kernels["moe_linear prefill (grouped)"] = {"ms": pre["moe_linear"], "rows": rows, "of_measured_tensor": moe_flops / (pre["moe_linear"] * 1e-3) / tens}
+        results.append(common(f"tibopel-w{width}", raw, r, kernels, {"experts": moe["router"]["experts"], "identity": moe["router"]["identity"], "top": top}))
+        results.append(_noganex_side(width, env))
+        results.append(_fetotar_latent_side(width, env))
+    return env["report"]("tibopel_compare", results)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1422,6 +1510,8 @@ def main():
                     help="Nasozen beside Noganex at equal size: prefill and decode throughput and per-kernel rooflines (one GPU)")
     ap.add_argument("--nomalorn-compare", action="store_true",
                     help="Nomalorn beside Noganex at equal size: prefill and decode throughput and per-kernel rooflines (one GPU)")
+    ap.add_argument("--tibopel-compare", action="store_true",
+                    help="Tibopel beside Noganex and Fetotar's latent attention at equal size: prefill and decode throughput and per-kernel rooflines (one GPU)")
     args = ap.parse_args()
     if args.warmup < 3:
         args.warmup = 3
@@ -1435,6 +1525,8 @@ def main():
         return run_nasozen_compare(args)
     if args.nomalorn_compare:
         return run_nomalorn_compare(args)
+    if args.tibopel_compare:
+        return run_tibopel_compare(args)
     workload = args.workload or DEFAULT_WORKLOAD
     if workload in MIXED_WORKLOADS:
         if args.impl == "reference":

@@ -112,8 +112,23 @@ def nomalorn_config(name: str) -> dict:
             "vocab": 32000, "width": W}
 
 
+def tibopel_config(name: str) -> dict:
+    """Three layers at the widths of the `noganex-w*` / `fetotar-w*` partners: attention (chunks of 2048, half of each head rotated, a gate
+    per head), latent attention (latent 512 + 64 rotated, sinks), attention again; each beside 16 squared-ReLU experts and 4 identity outputs of
+    which a token uses 2, and a shared expert (as many expert parameters as the partner's gated ones): raw config.json of the Tibopel family."""
+    W = {"tibopel-w2048": 2048, "tibopel-w4096": 4096}[name]
+    moe = {"kind": "moe", "expert": {"ff": W * 33 // 32}, "router": {"experts": 16, "identity": 4, "top": 2}, "shared": {"ff": W * 33 // 32}}
+    attn = {"dim": 128, "heads": W // 128, "kv_heads": W // 512, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 2048},
+            "rot": {"base": 1000000.0, "dims": 64, "scaling": {"factor": 8.0, "high": 4.0, "low": 1.0, "original": 4096}}}
+    latent = {"dim": 128, "heads": W // 128, "kv_rank": 512, "q_rank": 1536, "rot": {"base": 10000.0, "dims": 64}, "rot_dim": 64,
+              "scale": 192 ** -0.5, "vdim": 128}
+    layers = [{"type": "attention", "mixer": dict(attn), "mlp": dict(moe)}, {"type": "latent_attention", "mixer": latent, "mlp": dict(moe)},
+              {"type": "attention", "mixer": dict(attn), "mlp": dict(moe)}]
+    return {"architecture": "Tibopel", "layers": layers, "logit_softcap": 30.0, "norm": {"eps": 1e-5}, "vocab": 32000, "width": W}
+
+
 class SyntheticHybridWeights:
-    """Seeded random tensors of a Fetotar, Dubesun, Noganex, Nasozen or Nomalorn configuration, generated on the device by name (the `get_tensor`
+    """Seeded random tensors of a Fetotar, Dubesun, Noganex, Nasozen, Nomalorn or Tibopel configuration, generated on the device by name (the `get_tensor`
     side of `Weights`)."""
 
     def __init__(self, raw_config: dict, device, dtype, process_group, seed: int = 1234):
@@ -125,6 +140,8 @@ class SyntheticHybridWeights:
             from ..models.custom_modeling.nasozen_modeling import tensor_shapes
         elif raw_config.get("architecture") == "Nomalorn":
             from ..models.custom_modeling.nomalorn_modeling import tensor_shapes
+        elif raw_config.get("architecture") == "Tibopel":
+            from ..models.custom_modeling.tibopel_modeling import tensor_shapes
         else:
             from ..models.custom_modeling.fetotar_modeling import tensor_shapes
         self.shapes, self.device, self.dtype, self.process_group, self.seed = tensor_shapes(raw_config), device, dtype, process_group, seed
@@ -147,6 +164,8 @@ class SyntheticHybridWeights:
             t = torch.rand(shape, generator=gen, device=self.device) * 2.0 - 2.0
         elif leaf == "mix.f.b":
             t = torch.full(shape, 3.0, device=self.device)
+        elif leaf in ("mlp.correction", "mix.sink"):
+            t = torch.zeros(shape, device=self.device)
         elif leaf.endswith(".b") or (self.offset_norms and (leaf == "norm1" or name == "final.norm")):
             t = torch.zeros(shape, device=self.device)   # biases, and norm weights that are stored around zero
         elif leaf in ("mix.lq1", "mix.lk1", "mix.lq2", "mix.lk2"):
