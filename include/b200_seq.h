@@ -43,19 +43,20 @@ int b200_seq_ff_clamped_gate(const void* gu, void* out, int dt, int64_t rows, in
 int b200_seq_side_gate(const float* a, const int64_t* ids, const void* table, int64_t ld_table, int64_t col0, int dim, int64_t V, void* out,
                        int dt, int64_t rows, void* stream);
 int b200_seq_rms_add(const float* y, const void* w, int dt, float* resid, int64_t T, int64_t W, float eps, void* stream);
-/* cache row of every token = [unit_rms(latent) * w | rotated key part]; q_abs[:, :, R:] = rotated query parts */
-int b200_seq_latent_prepare(const float* down, int64_t ld_down, int col_c, int col_kr, const float* q, int64_t ld_q, int q_head_stride,
+/* cache row of every token = [unit_rms(latent) * w | rotated key part]; q_abs[:, :, R:] = rotated query parts (q, q_abs of type dt) */
+int b200_seq_latent_prepare(const float* down, int64_t ld_down, int col_c, int col_kr, const void* q, int64_t ld_q, int q_head_stride,
                             int q_rot_off, const void* cnorm_w, const float* cos_t, const float* sin_t, const int64_t* position_ids,
-                            const int64_t* slot_mapping, void* cache, int dt, float* q_abs, int64_t T, int H, int R, int r, int rot_dims,
+                            const int64_t* slot_mapping, void* cache, int dt, void* q_abs, int64_t T, int H, int R, int r, int rot_dims,
                             float eps, void* stream);
-/* out[t, h, :R] = sum_j softmax_j((q_abs[t, h] . cache_row(j)) * scale) cache_row(j)[:R], j over (p - window, p] of t's sequence.
+/* out[t, h, :R] = sum_j softmax_j((q_abs[t, h] . cache_row(j)) * scale) cache_row(j)[:R], j over (p - window, p] of t's sequence;
+ * q_abs, cache and out of type dt.
  * b200_seq_latent_attn_splits: over how many blocks the tensor-core kernel should split each token's keys for this shape (0: the
  * shape takes the plain kernel) and the fp32 workspace (`partial`) that takes; partial NULL / nsplit <= 1: no split.  sink fp32 [H]
  * (NULL: none): exp(sink[h]) joins head h's soft-max denominator (unscaled) and carries no value */
-int b200_seq_latent_attn_splits(int dt, int64_t Tq, int H, int R, int r, int64_t* workspace_floats);
-int b200_seq_latent_attn(const float* q_abs, const void* cache, int dt, const int32_t* block_table, int64_t bt_stride,
-                         const int32_t* seq_of_token, const int64_t* position_ids, float* out, int64_t Tq, int H, int R, int r, int window,
-                         float scale, int page, float* partial, int nsplit, const float* sink, void* stream);
+int b200_seq_latent_attn_splits(int dt, int64_t Tq, int B, int H, int R, int r, int64_t* workspace_floats);
+int b200_seq_latent_attn(const void* q_abs, const void* cache, int dt, const int32_t* block_table, int64_t bt_stride,
+                         const int32_t* seq_of_token, const int32_t* cu_q, int B, const int64_t* position_ids, void* out, int64_t Tq, int H, int R,
+                         int r, int window, float scale, int page, float* partial, int nsplit, const float* sink, void* stream);
 /* SiLU(depth-wise causal convolution) of columns [col0, col0 + C) of u; conv_state [slots, taps - 1, C] read and advanced */
 int b200_seq_causal_conv_silu(const float* u, int64_t ld_u, int col0, int C, int taps, const void* w, const void* bias, int dt,
                               float* conv_state, const int32_t* state_slots, const int32_t* seq_of_token, const int32_t* cu_q,
@@ -119,6 +120,18 @@ int b200_seq_moe_route_scored(const float* logits, int64_t ld, int64_t T, int E,
                               float weight_scale, int32_t* ids, float* weights, int32_t* plan, void* stream);
 /* the plan's row_of [T, top]: compact row of every pick, -1 for an identity output */
 int32_t* b200_seq_moe_row_of(int32_t* plan, int64_t T, int E, int top);
+/* the plan's offsets [E + 1]: first compact row of every expert, then their number */
+int32_t* b200_seq_moe_offsets(int32_t* plan, int64_t T, int E, int top);
+/* groups of bfloat16 products on tcgen05 tensor cores, one launch each.
+ * heads: Y[t, z, :N] = W[z] X[t, z, :K]; token strides ldx / ldy and head strides head_x / head_y in elements (Y may be a slice of wider
+ * rows), W [Z, N, K] dense; K, ldx, head_x multiples of 8.
+ * experts: Y[row] = act(W[expert(row)] X[row]) over a plan's compact rows, X [max_rows, K], Y [max_rows, N] and W [E, N, K] dense; act 0:
+ * none, 1: relu(z)^2.  gave_up: blocks that gave up a bounded wait (0 unless something is wrong) */
+int b200_seq_heads_gemm(const void* x, int64_t ldx, int64_t head_x, const void* w, void* y, int y_dt, int64_t ldy, int64_t head_y, int64_t T,
+                        int64_t Z, int64_t N, int64_t K, void* stream);
+int b200_seq_experts_gemm(const void* x, const void* w, void* y, int y_dt, const int32_t* offsets, int64_t max_rows, int E, int64_t N, int64_t K,
+                          int act, void* stream);
+int b200_seq_group_gemm_gave_up(void);
 /* resid (fp32) += v / sqrt(mean v^2 + eps) * w, v = y * sigmoid(gate) (gate NULL: y); typed (type dt, may be NULL) = the updated rows */
 int b200_seq_gated_rms_add(const float* y, const float* gate, const void* w, int dt, float* resid, void* typed, int64_t T, int64_t W, float eps,
                            void* stream);

@@ -255,6 +255,7 @@ def test_latent_attention_window_edges_page_borders_and_far_keys(dtype, R, r):
         for i, (p, j) in enumerate(pairs):
             if 0 <= j <= p:
                 q_abs[i, i % H] += 6.0 * rows[j].float() / rows[j].float().norm() ** 2 * 8.0
+        q_abs = q_abs.to(dtype).float()
         ref = _attn_reference(q_abs, rows.float(), list(range(L)), [0] * L, q_pos, [0] * len(pairs), R, w, scale)
         cache = torch.zeros(32, 16, D, dtype=dtype, device=DEV)
         cache.view(-1, D)[:L] = rows.to(DEV)
@@ -263,13 +264,13 @@ def test_latent_attention_window_edges_page_borders_and_far_keys(dtype, R, r):
         for i, p in enumerate(q_pos):
             st = _step([(p, 1)], 32)
             st.block_table = full.block_table
-            got = ops.latent_attn(q_abs[i:i + 1].to(DEV).contiguous(), cache, st, R, r, win, scale).cpu().double()
+            got = ops.latent_attn(q_abs[i:i + 1].to(dtype).to(DEV).contiguous(), cache, st, R, r, win, scale).cpu().double()
             assert torch.allclose(got, ref[i:i + 1], atol=1e-4 if dtype == torch.float32 else 3e-2), (far, pairs[i])
         # and all positions of the sequence as one prompt: row p is query p
         qs = torch.randn(L, H, D, generator=g) * 0.2
         for i, (p, j) in enumerate(pairs):
             qs[p] = q_abs[i]
-        got = ops.latent_attn(qs.to(DEV).contiguous(), cache, full, R, r, win, scale).cpu().double()
+        got = ops.latent_attn(qs.to(dtype).to(DEV).contiguous(), cache, full, R, r, win, scale).cpu().double()
         for p, i in {p: i for i, p in enumerate(q_pos)}.items():  # a position listed twice carries its last query
             assert torch.allclose(got[p], ref[i], atol=1e-4 if dtype == torch.float32 else 3e-2), (far, "prompt", pairs[i])
 

@@ -137,8 +137,8 @@ SEQ_SIGNATURES = {
     "b200_seq_side_gate": (_I, [_P, _P, _P, _L, _L, _I, _L, _P, _I, _L, _P]),
     "b200_seq_rms_add": (_I, [_P, _P, _I, _P, _L, _L, _F, _P]),
     "b200_seq_latent_prepare": (_I, [_P, _L, _I, _I, _P, _L, _I, _I, _P, _P, _P, _P, _P, _P, _I, _P, _L, _I, _I, _I, _I, _F, _P]),
-    "b200_seq_latent_attn_splits": (_I, [_I, _L, _I, _I, _I, ctypes.POINTER(c_int64)]),
-    "b200_seq_latent_attn": (_I, [_P, _P, _I, _P, _L, _P, _P, _P, _L, _I, _I, _I, _I, _F, _I, _P, _I, _P, _P]),
+    "b200_seq_latent_attn_splits": (_I, [_I, _L, _I, _I, _I, _I, ctypes.POINTER(c_int64)]),
+    "b200_seq_latent_attn": (_I, [_P, _P, _I, _P, _L, _P, _P, _I, _P, _P, _L, _I, _I, _I, _I, _F, _I, _P, _I, _P, _P]),
     "b200_seq_causal_conv_silu": (_I, [_P, _L, _I, _I, _I, _P, _P, _I, _P, _P, _P, _P, _P, _P, _L, _I, _P]),
     "b200_seq_ssm_scan": (_I, [_P, _L, _I, _I, _I, _P, _L, _I, _P, _P, _P, _I, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P]),
     "b200_seq_mlstm_scan": (_I, [_P, _L, _I, _I, _I, _I, _I, _P, _P, _I, _F, _F, _P, _P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _P]),
@@ -156,6 +156,10 @@ SEQ_SIGNATURES = {
     "b200_seq_moe_combine_add": (_I, [_P, _P, _P, _L, _P, _P, _L, _I, _I, _L, _P]),
     "b200_seq_moe_route_scored": (_I, [_P, _L, _L, _I, _I, _I, _I, _P, _I, _F, _P, _P, _P, _P]),
     "b200_seq_moe_row_of": (_P, [_P, _L, _I, _I]),
+    "b200_seq_moe_offsets": (_P, [_P, _L, _I, _I]),
+    "b200_seq_heads_gemm": (_I, [_P, _L, _L, _P, _P, _I, _L, _L, _L, _L, _L, _L, _P]),
+    "b200_seq_experts_gemm": (_I, [_P, _P, _P, _I, _P, _L, _I, _L, _L, _I, _P]),
+    "b200_seq_group_gemm_gave_up": (_I, []),
     "b200_seq_gated_rms_add": (_I, [_P, _P, _P, _I, _P, _P, _L, _L, _F, _P]),
     "b200_seq_cast_rows": (_I, [_P, _P, _I, _L, _P]),
     "b200_seq_ff_gate": (_I, [_P, _P, _I, _L, _L, _I, _P]),

@@ -419,6 +419,8 @@ extern "C" int64_t b200_seq_moe_plan_ints(int64_t T, int E, int top) {
 
 extern "C" int32_t* b200_seq_moe_row_of(int32_t* plan, int64_t T, int E, int top) { return moe_plan_view(plan, T, E, top).row_of; }
 
+extern "C" int32_t* b200_seq_moe_offsets(int32_t* plan, int64_t T, int E, int top) { return moe_plan_view(plan, T, E, top).offsets; }
+
 // logits fp32 [T, E_all] (leading dimension ld) -> ids int32 [T, top], weights fp32 [T, top] and the plan (b200_seq_moe_plan_ints(T, E, top)
 // int32 values) over the E experts; the router outputs E .. E_all - 1 are identity outputs.
 // mode 0: soft-max over the picked logits (correction, weight_scale unused); mode 1 / 2: scores sigmoid(logit) / soft-max over all E_all

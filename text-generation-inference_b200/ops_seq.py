@@ -99,11 +99,17 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
 
 
 def linear_per_head(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-    """x [M, Z, K], w [Z, N, K], out [M, Z, N] (all may be slices with a wider last-but-one stride): out[:, z] = x[:, z] @ w[z]^T."""
+    """x [M, Z, K], w [Z, N, K], out [M, Z, N] (all may be slices with a wider last-but-one stride): out[:, z] = x[:, z] @ w[z]^T.
+    bfloat16 operands with K and strides in multiples of 8 go to the tcgen05 groups (csrc/seq_group_gemm.cu)."""
     _cuda(x, w, out)
     M, Z, K = x.shape
     N = w.shape[1]
     assert w.shape == (Z, N, K) and out.shape == (M, Z, N) and x.stride(2) == 1 and w.stride(2) == 1 and out.stride(2) == 1
+    if (_TC_GEMM and x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and K % 8 == 0 and x.stride(0) % 8 == 0 and x.stride(1) % 8 == 0
+            and w.is_contiguous() and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0 and x.stride(0) >= (Z - 1) * x.stride(1) + K):
+        _lib.check_seq(_lib.load_seq().b200_seq_heads_gemm(_ptr(x), x.stride(0), x.stride(1), _ptr(w), _ptr(out), _dt(out), out.stride(0), out.stride(1),
+                                                           M, Z, N, K, _stream()), "seq_heads_gemm")
+        return out
     _lib.check_seq(_lib.load_seq().b200_seq_linear(_ptr(x), _dt(x), x.stride(0), x.stride(1), _ptr(w), _dt(w), w.stride(1), w.stride(0), None,
                                                    _ptr(out), _dt(out), out.stride(0), out.stride(1), M, N, K, Z, _stream()), "seq_linear")
     return out
@@ -194,9 +200,10 @@ def token_side(residual: torch.Tensor, residual_typed: torch.Tensor, ids: torch.
 def latent_prepare(down: torch.Tensor, col_c: int, col_kr: int, q: torch.Tensor, q_head_stride: int, q_rot_off: int,
                    cnorm_w: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, step: RaggedStep, cache: torch.Tensor, q_abs: torch.Tensor,
                    H: int, R: int, r: int, rot_dims: int, eps: float) -> None:
-    """Writes each token's cache row [unit_rms(latent) * w | rotated key part] and the rotated query parts q_abs[:, :, R:]."""
+    """Writes each token's cache row [unit_rms(latent) * w | rotated key part] and the rotated query parts q_abs[:, :, R:].  down fp32; q and
+    q_abs have the cache's element type."""
     _cuda(down, q, cache, q_abs)
-    assert down.dtype == torch.float32 and q.dtype == torch.float32 and q_abs.dtype == torch.float32 and cos.dtype == torch.float32
+    assert down.dtype == torch.float32 and q.dtype == cache.dtype and q_abs.dtype == cache.dtype and cos.dtype == torch.float32
     assert q_abs.is_contiguous() and cache.is_contiguous() and cos.is_contiguous() and sin.is_contiguous()
     _lib.check_seq(_lib.load_seq().b200_seq_latent_prepare(
         _ptr(down), down.stride(0), col_c, col_kr, _ptr(q), q.stride(0), q_head_stride, q_rot_off, _ptr(cnorm_w), _ptr(cos), _ptr(sin),
@@ -206,21 +213,21 @@ def latent_prepare(down: torch.Tensor, col_c: int, col_kr: int, q: torch.Tensor,
 
 def latent_attn(q_abs: torch.Tensor, cache: torch.Tensor, step: RaggedStep, R: int, r: int, window: int, scale: float,
                 sink: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """q_abs fp32 [T, H, R + r], cache [blocks, page, R + r] -> fp32 [T, H, R]: soft-max attention of every token over the cache
+    """q_abs [T, H, R + r], cache [blocks, page, R + r] of one element type -> [T, H, R] in it: soft-max attention of every token over the cache
     rows of its own sequence at positions (p - window, p], in latent space (window 0: all of
     them).  sink fp32 [H]: exp(sink[h]) joins head h's soft-max denominator (not scaled) and carries no value."""
     _cuda(q_abs, cache, sink)
     T, H, D = q_abs.shape
     assert sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.shape == (H,))
-    assert D == R + r and cache.shape[-1] == D and q_abs.is_contiguous() and cache.is_contiguous()
-    out = torch.empty(T, H, R, dtype=torch.float32, device=q_abs.device)
+    assert D == R + r and cache.shape[-1] == D and q_abs.is_contiguous() and cache.is_contiguous() and q_abs.dtype == cache.dtype
+    out = torch.empty(T, H, R, dtype=q_abs.dtype, device=q_abs.device)
     lib = _lib.load_seq()
     need = ctypes.c_int64(0)
-    nsplit = lib.b200_seq_latent_attn_splits(_dt(cache), T, H, R, r, ctypes.byref(need)) if _ATTN_SPLIT else 1
+    nsplit = lib.b200_seq_latent_attn_splits(_dt(cache), T, step.B, H, R, r, ctypes.byref(need)) if _ATTN_SPLIT else 1
     partial = torch.empty(need.value, dtype=torch.float32, device=q_abs.device) if nsplit > 1 else None
     _lib.check_seq(lib.b200_seq_latent_attn(
-        _ptr(q_abs), _ptr(cache), _dt(cache), _ptr(step.block_table), step.block_table.stride(0), _ptr(step.seq_of_token),
-        _ptr(step.position_ids), _ptr(out), T, H, R, r, int(window), float(scale), cache.shape[1], _ptr(partial), nsplit, _ptr(sink),
+        _ptr(q_abs), _ptr(cache), _dt(cache), _ptr(step.block_table), step.block_table.stride(0), _ptr(step.seq_of_token), _ptr(step.cu_q),
+        step.B, _ptr(step.position_ids), _ptr(out), T, H, R, r, int(window), float(scale), cache.shape[1], _ptr(partial), nsplit, _ptr(sink),
         _stream()), "seq_latent_attn")
     return out
 
@@ -414,9 +421,18 @@ def moe_gather_rows(a: torch.Tensor, r: MoeRouting) -> torch.Tensor:
     return out
 
 
-def moe_expert_offsets(r: MoeRouting) -> list:
-    """first compact row of every expert, and the row count at the end (a device-to-host read: not inside a captured graph)"""
-    return r.plan[r.experts:2 * r.experts + 1].tolist()
+def experts_linear(a: torch.Tensor, w: torch.Tensor, r: MoeRouting, out_dtype: torch.dtype, act: int = ACT_NONE) -> torch.Tensor:
+    """moe_linear over compact rows for steps of many rows per expert: bfloat16 a [T * top, K] (as moe_gather_rows leaves them) and w [E, N, K] on
+    tcgen05 tensor cores, one launch for any distribution of the rows; K % 8 == 0."""
+    _cuda(a, w)
+    E, N, K = w.shape
+    assert a.dtype == w.dtype == torch.bfloat16 and a.is_contiguous() and w.is_contiguous() and a.shape == (r.T * r.top, K) and E == r.experts
+    assert act in (ACT_NONE, ACT_RELU2)
+    out = torch.empty(r.T * r.top, N, dtype=out_dtype, device=a.device)
+    lib = _lib.load_seq()
+    _lib.check_seq(lib.b200_seq_experts_gemm(_ptr(a), _ptr(w), _ptr(out), _dt(out), lib.b200_seq_moe_offsets(_ptr(r.plan), r.T, E, r.top), r.T * r.top, E,
+                                             N, K, int(act == ACT_RELU2), _stream()), "seq_experts_gemm")
+    return out
 
 
 def moe_combine_add(resid: torch.Tensor, mix: Optional[torch.Tensor], y: Optional[torch.Tensor], r: Optional[MoeRouting]) -> None:

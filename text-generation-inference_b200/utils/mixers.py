@@ -117,18 +117,17 @@ class LatentAttention(nn.Module):
         T = step.T
         down = ops.linear(h, self.w_in, out_dtype=torch.float32)
         cq = ops.group_rmsnorm_gate(down[:, :Q], self.dq_norm, 1, self.eps, self.dtype)
-        q = ops.linear(cq, self.w_uq, out_dtype=torch.float32)
-        q_abs = torch.empty(T, H, R + r, dtype=torch.float32, device=h.device)
+        q = ops.linear(cq, self.w_uq)
+        q_abs = torch.empty(T, H, R + r, dtype=self.dtype, device=h.device)
         cos, sin = self.rotary.tables(max_s, h.device)
         ops.latent_prepare(down, Q, Q + R, q, d + r, d, self.dkv_norm, cos, sin, step, store, q_abs, H, R, r, self.rotary.dims, self.eps)
         ops.linear_per_head(q.view(T, H, d + r)[:, :, :d], self.w_uk_t, q_abs[:, :, :R])
         o_lat = ops.latent_attn(q_abs, store, step, R, r, self.window, self.scale, self.sink)
-        o = torch.empty(T, H, dv, dtype=torch.float32, device=h.device)
+        o = torch.empty(T, H, dv, dtype=torch.float32 if self.gate else self.dtype, device=h.device)
         ops.linear_per_head(o_lat, self.w_uv, o)
+        o = o.view(T, H * dv)
         if self.gate:
-            o = ops.group_rmsnorm_gate(o.view(T, H * dv), None, 0, self.eps, self.dtype, gate=down[:, Q + R + r:], gate_kind=ops.GATE_SIGMOID_AFTER)
-        else:
-            o = ops.cast_rows(o.view(T, H * dv), self.dtype)
+            o = ops.group_rmsnorm_gate(o, None, 0, self.eps, self.dtype, gate=down[:, Q + R + r:], gate_kind=ops.GATE_SIGMOID_AFTER)
         return ops.linear(o, self.w_o, out_dtype=self.out_dtype)
 
 
@@ -330,7 +329,7 @@ class RoutedExperts(nn.Module):
     products of the same input that run with the router's; `route` returns their fp32 results after the routing.
     Tensors under `prefix`: router, [correction,] [e<j>.gate,] e<j>.up, e<j>.down."""
 
-    dense_rows_per_expert = 64   # average rows per expert from which a step runs one dense product per expert
+    group_rows_per_expert = 64   # average rows per expert from which a step takes the tcgen05 groups
 
     def __init__(self, prefix: str, weights, *, experts: int, top: int, limit: Optional[float], alpha: float = 1.702,
                  sigmoid_scores: bool = False, correction: bool = False, weight_scale: float = 1.0, softmax_scores: bool = False,
@@ -372,21 +371,10 @@ class RoutedExperts(nn.Module):
     def experts(self, h: torch.Tensor, routing) -> torch.Tensor:
         act1 = ops.ACT_RELU2 if self.plain else ops.ACT_NONE
         rows = h.shape[0] * self.top
-        if h.dtype == torch.bfloat16 and rows >= self.dense_rows_per_expert * self.E and not torch.cuda.is_current_stream_capturing():
-            # prompts: enough rows per expert for the tcgen05 product (ops.linear) to pay - one product per expert over its run of
-            # compact rows; the runs' bounds are read back once per layer, so this form stays out of captured decode graphs
-            offs = ops.moe_expert_offsets(routing)
-            a = ops.moe_gather_rows(h, routing)
-            gu = torch.empty(rows, self.w_gate_up.shape[1], dtype=h.dtype, device=h.device)
-            for e in range(self.E):
-                if offs[e + 1] > offs[e]:
-                    ops.linear(a[offs[e]:offs[e + 1]], self.w_gate_up[e], out=gu[offs[e]:offs[e + 1]], act=act1)
-            act = self._act(gu)
-            y = torch.empty(rows, self.w_down.shape[1], dtype=torch.float32, device=h.device)
-            for e in range(self.E):
-                if offs[e + 1] > offs[e]:
-                    ops.linear(act[offs[e]:offs[e + 1]], self.w_down[e], out=y[offs[e]:offs[e + 1]])
-            return y
+        if h.dtype == torch.bfloat16 and rows >= self.group_rows_per_expert * self.n_route and h.shape[1] % 8 == 0 and self.w_down.shape[2] % 8 == 0:
+            # prompts: enough rows per expert for the tcgen05 products, one launch each over the compact rows of all experts
+            gu = ops.experts_linear(ops.moe_gather_rows(h, routing), self.w_gate_up, routing, h.dtype, act=act1)
+            return ops.experts_linear(self._act(gu), self.w_down, routing, torch.float32)
         gu = ops.moe_linear(h, self.w_gate_up, routing, gather=True, out_dtype=h.dtype, act=act1)
         return ops.moe_linear(self._act(gu), self.w_down, routing, gather=False, out_dtype=torch.float32)
 
