@@ -694,6 +694,11 @@ def _by_op(log):
     return out
 
 
+def _products_ms(ops):
+    """projections and the experts' grouped products of one step"""
+    return ops["linear"] + ops.get("experts_linear", 0.0)
+
+
 def _traced_decode_step(model, batch, lib):
     """device time of every kernel of one fused decode step: the step is captured in a graph of its own with a time stamp after
     every launch of the library (host latency is out of the picture, L2 as in the served step).  -> ({kernel: us}, total us)"""
@@ -992,7 +997,7 @@ def run_dubesun_compare(args):
             prefill_once()
         pre_ms = timed(prefill_once, K)
         names = ["linear", "embed_add_pos", "rmsnorm_rows", "causal_conv", "heads_prepare", "paged_attn", "diff_combine", "group_rmsnorm_gate",
-                 "moe_route", "moe_gather_rows", "moe_linear", "ff_clamped_gate", "moe_combine_add"]
+                 "moe_route", "moe_gather_rows", "experts_linear", "moe_linear", "ff_clamped_gate", "moe_combine_add"]
         log = []
         saved = _timed_ops(ops_seq, names, log)
         prefill_once()
@@ -1051,7 +1056,7 @@ def run_dubesun_compare(args):
             "paged_attn prefill (3 layers)": {"ms": pre_ops["paged_attn"], "tflops": attn_flops / pre_ops["paged_attn"] / 1e9,
                                               "of_measured_tensor": attn_flops / (pre_ops["paged_attn"] * 1e-3) / tens},
             "paged_attn decode (3 layers)": {"us": attn_us, "of_measured_hbm": DB * ctx * attn_rows * 2 / (max(attn_us, 1e-9) * 1e-6) / hbm},
-            "linear prefill (projections + one product per expert)": {"ms": pre_ops["linear"], "of_measured_tensor": lin_flops / (pre_ops["linear"] * 1e-3) / tens},
+            "linear prefill (projections + experts)": {"ms": _products_ms(pre_ops), "of_measured_tensor": lin_flops / (_products_ms(pre_ops) * 1e-3) / tens},
             "moe_linear decode (grouped, picked experts' weights once)": {"us": moe_us, "experts_picked_all_layers": picked, "of_measured_hbm":
                                                                           picked * expert_w * 2 / (max(moe_us, 1e-9) * 1e-6) / hbm},
             "linear decode (tcgen05 projections)": {"us": dec_k.get("gemm_f16_kernel", 0.0), "of_measured_hbm":
@@ -1153,7 +1158,7 @@ def _noganex_side(width, env):
     timed, lib, hbm, tens, common, us = (env[k] for k in ("timed", "lib", "hbm", "tens", "common", "us"))
     raw = noganex_config(f"noganex-w{width}")
     names = ["linear", "embed_scale", "cast_rows", "rmsnorm_rows", "gated_rms_add", "causal_conv", "delta_scan", "qk_rot_prepare", "talk_attn",
-             "group_rmsnorm_gate", "moe_route", "moe_gather_rows", "moe_linear", "ff_gate", "moe_combine_add"]
+             "group_rmsnorm_gate", "moe_route", "moe_gather_rows", "experts_linear", "moe_linear", "ff_gate", "moe_combine_add"]
     r = _stream_family_measure(raw, noganex_modeling.NoganexConfig(raw), names, PB, PL, DB, DL, K, Wm, timed, lib)
     shapes = noganex_modeling.tensor_shapes(raw)
     attn = [l["mixer"] for l in raw["layers"] if l["type"] == "attention"]
@@ -1175,8 +1180,8 @@ def _noganex_side(width, env):
         "talk_attn decode": {"us": a_us, "of_measured_hbm": DB * ctx * attn_row * 2 / (max(a_us, 1e-9) * 1e-6) / hbm},
         "delta_scan prefill": {"ms": r["pre_ops"]["delta_scan"], "tokens_per_s_per_layer": PB * PL * len(delta) / (r["pre_ops"]["delta_scan"] * 1e-3)},
         "delta_scan decode": {"us": s_us, "of_measured_hbm": DB * state_b / (max(s_us, 1e-9) * 1e-6) / hbm},
-        "linear prefill (projections, gates, one product per expert)": {"ms": r["pre_ops"]["linear"],
-                                                                        "of_measured_tensor": lin_flops / (r["pre_ops"]["linear"] * 1e-3) / tens},
+        "linear prefill (projections, gates, experts)": {"ms": _products_ms(r["pre_ops"]),
+                                                                        "of_measured_tensor": lin_flops / (_products_ms(r["pre_ops"]) * 1e-3) / tens},
         "moe_linear decode (grouped, picked experts' weights once)": {"us": m_us, "experts_picked_all_layers": r["picked"], "of_measured_hbm":
                                                                       r["picked"] * expert_w * 2 / (max(m_us, 1e-9) * 1e-6) / hbm},
         "linear decode (tcgen05 projections)": {"us": g_us, "of_measured_hbm": (dense_w + head_w) * 2 / (max(g_us, 1e-9) * 1e-6) / hbm},
@@ -1254,7 +1259,7 @@ def run_noganex_compare(args):
         # ---------------------------------------------------------------- Dubesun, the partner
         raw = dubesun_config(f"dubesun-w{width}")
         names = ["linear", "embed_add_pos", "rmsnorm_rows", "causal_conv", "heads_prepare", "paged_attn", "diff_combine", "group_rmsnorm_gate",
-                 "moe_route", "moe_gather_rows", "moe_linear", "ff_clamped_gate", "moe_combine_add"]
+                 "moe_route", "moe_gather_rows", "experts_linear", "moe_linear", "ff_clamped_gate", "moe_combine_add"]
         r = _stream_family_measure(raw, dubesun_modeling.DubesunConfig(raw), names, PB, PL, DB, DL, K, Wm, timed, lib)
         shapes = dubesun_modeling.tensor_shapes(raw)
         attn_flops, attn_row = 0, 0
@@ -1274,8 +1279,8 @@ def run_noganex_compare(args):
             "paged_attn prefill": {"ms": r["pre_ops"]["paged_attn"], "tflops": attn_flops / r["pre_ops"]["paged_attn"] / 1e9,
                                    "of_measured_tensor": attn_flops / (r["pre_ops"]["paged_attn"] * 1e-3) / tens},
             "paged_attn decode": {"us": a_us, "of_measured_hbm": DB * ctx * attn_row * 2 / (max(a_us, 1e-9) * 1e-6) / hbm},
-            "linear prefill (projections + one product per expert)": {"ms": r["pre_ops"]["linear"],
-                                                                      "of_measured_tensor": lin_flops / (r["pre_ops"]["linear"] * 1e-3) / tens},
+            "linear prefill (projections + experts)": {"ms": _products_ms(r["pre_ops"]),
+                                                                      "of_measured_tensor": lin_flops / (_products_ms(r["pre_ops"]) * 1e-3) / tens},
             "moe_linear decode (grouped, picked experts' weights once)": {"us": m_us, "experts_picked_all_layers": r["picked"], "of_measured_hbm":
                                                                           r["picked"] * expert_w * 2 / (max(m_us, 1e-9) * 1e-6) / hbm},
             "linear decode (tcgen05 projections)": {"us": g_us, "of_measured_hbm": (proj_w + head_w) * 2 / (max(g_us, 1e-9) * 1e-6) / hbm},
@@ -1300,7 +1305,7 @@ def run_nasozen_compare(args):
     for width in env["widths"]:
         raw = nasozen_config(f"nasozen-w{width}")
         names = ["linear", "embed_scale", "streams_step", "causal_conv", "qk_rot_prepare", "talk_attn", "heads_turn_gate", "mingru_scan", "mlstm_scan",
-                 "gdelta_scan", "group_rmsnorm_gate", "ff_act", "moe_route", "moe_gather_rows", "moe_linear", "ff_gate", "moe_combine_add"]
+                 "gdelta_scan", "group_rmsnorm_gate", "ff_act", "moe_route", "moe_gather_rows", "experts_linear", "moe_linear", "ff_gate", "moe_combine_add"]
         cfg = nasozen_modeling.NasozenConfig(raw)
         r = _stream_family_measure(raw, cfg, names, PB, PL, DB, DL, K, Wm, timed, lib)
         shapes = nasozen_modeling.tensor_shapes(raw)
@@ -1339,8 +1344,8 @@ def run_nasozen_compare(args):
             "streams_step prefill": {"ms": r["pre_ops"]["streams_step"], "of_measured_hbm": T * stream_b / (r["pre_ops"]["streams_step"] * 1e-3) / hbm},
             "streams_step decode": {"us": us(dk, "streams_step"), "launches": subs + 1,
                                     "of_measured_hbm": DB * stream_b / (max(us(dk, "streams_step"), 1e-9) * 1e-6) / hbm},
-            "linear prefill (projections, one product per expert)": {"ms": r["pre_ops"]["linear"],
-                                                                     "of_measured_tensor": lin_flops / (r["pre_ops"]["linear"] * 1e-3) / tens},
+            "linear prefill (projections, experts)": {"ms": _products_ms(r["pre_ops"]),
+                                                                     "of_measured_tensor": lin_flops / (_products_ms(r["pre_ops"]) * 1e-3) / tens},
             "moe_linear decode (grouped, picked experts' weights once)": {"us": m_us, "experts_picked_all_layers": r["picked"], "of_measured_hbm":
                                                                           r["picked"] * expert_w * 2 / (max(m_us, 1e-9) * 1e-6) / hbm},
             "linear decode (tcgen05 projections)": {"us": g_us, "of_measured_hbm": (dense_w + head_w) * 2 / (max(g_us, 1e-9) * 1e-6) / hbm},
@@ -1447,7 +1452,7 @@ def run_tibopel_compare(args):
     for width in env["widths"]:
         raw = tibopel_config(f"tibopel-w{width}")
         names = ["linear", "linear_per_head", "embed_scale", "halves_step", "qk_rot_prepare", "talk_attn", "heads_turn_gate", "group_rmsnorm_gate",
-                 "latent_prepare", "latent_attn", "cast_rows", "moe_route", "moe_gather_rows", "moe_linear", "ff_act", "rmsnorm_rows", "soft_cap"]
+                 "latent_prepare", "latent_attn", "cast_rows", "moe_route", "moe_gather_rows", "experts_linear", "moe_linear", "ff_act", "rmsnorm_rows", "soft_cap"]
         r = _stream_family_measure(raw, tibopel_modeling.TibopelConfig(raw), names, PB, PL, DB, DL, K, Wm, timed, lib)
         shapes, L = tibopel_modeling.tensor_shapes(raw), raw["layers"]
         attn = [l["mixer"] for l in L if l["type"] == "attention"]
@@ -1463,8 +1468,6 @@ def run_tibopel_compare(args):
         # the picks that are experts (identity outputs cost nothing): counted in the prefill that was timed
         rows = r["pre_rows"]
         lin_flops, moe_flops = 2 * T * dense_w + 2 * PB * head_w, 2 * rows * expert_w
-        if "moe_linear" not in pre:      # one dense product per expert: inside `linear`
-            lin_flops, moe_flops = lin_flops + moe_flops, 0
         # a layer's boundary: stream in and out, the mixer's and the shared expert's results, the picked rows, the passed row, two typed rows out
         stream_b = sum(width * (8 + 4 + 4 + 4 * top + 2 + 4) for _ in L)
         a_us, m_us, g_us, h_us = us(dk, "talk_attn"), us(dk, "moe_linear"), dk.get("gemm_f16_kernel", 0.0), us(dk, "halves_step")
@@ -1480,8 +1483,8 @@ def run_tibopel_compare(args):
             "halves_step prefill": {"ms": pre["halves_step"], "of_measured_hbm": T * stream_b / (pre["halves_step"] * 1e-3) / hbm},
             "halves_step decode": {"us": h_us, "launches": len(L) + 1, "of_measured_hbm": DB * stream_b / (max(h_us, 1e-9) * 1e-6) / hbm},
         }
-        if moe_flops:
-            kernels["moe_linear prefill (grouped)"] = {"ms": pre["moe_linear"], "rows": rows, "of_measured_tensor": moe_flops / (pre["moe_linear"] * 1e-3) / tens}
+        kernels["experts_linear prefill (grouped)"] = {"ms": pre["experts_linear"], "rows": rows,
+                                                       "of_measured_tensor": moe_flops / (pre["experts_linear"] * 1e-3) / tens}
         results.append(common(f"tibopel-w{width}", raw, r, kernels, {"experts": moe["router"]["experts"], "identity": moe["router"]["identity"], "top": top}))
         results.append(_noganex_side(width, env))
         results.append(_fetotar_latent_side(width, env))

@@ -15,6 +15,7 @@ Checkpoint naming: `embed`, `l<i>.norm1|norm2`, `l<i>.mix.*`, `l<i>.mlp.*`, `fin
 """
 from __future__ import annotations
 
+import copy
 import math
 from typing import Dict, List, Optional
 
@@ -196,7 +197,7 @@ def random_config(*, width: int = 40, vocab: int = 72, order=("attention", "late
                  "shared": {"ff": shared} if shared else None}
         layer = {"type": kind, "mixer": m, "mlp": f}
         if i < len(shares) and shares[i] is not None:
-            layer = {**layers[shares[i]], "weights_of": shares[i]}
+            layer = {**copy.deepcopy(layers[shares[i]]), "weights_of": shares[i]}
         layers.append(layer)
     cfg = {"architecture": "Tibopel", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width}
     if cap:
