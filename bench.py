@@ -704,7 +704,9 @@ def _traced_decode_step(model, batch, lib):
     every launch of the library (host latency is out of the picture, L2 as in the served step).  -> ({kernel: us}, total us)"""
     import re
     import torch
+    from tgis_b200 import ops_seq
     cap = 4096
+    beside, ops_seq.SIDE_STREAM = ops_seq.SIDE_STREAM, False   # stamps follow one stream: nothing runs side by side in the traced step
     buf = torch.zeros(cap, dtype=torch.int64, device=model.device)
     side = torch.cuda.Stream()
     side.wait_stream(torch.cuda.current_stream())
@@ -721,6 +723,7 @@ def _traced_decode_step(model, batch, lib):
             g.replay()
         side.synchronize()
     torch.cuda.current_stream().wait_stream(side)
+    ops_seq.SIDE_STREAM = beside
     names = names_buf.value.decode().strip().split("\n")
     t = buf[:n].cpu().tolist()
     out = {}

@@ -657,3 +657,39 @@ def test_replayed_trace_writes_the_reference_logits(tmp_path):
         for i, ref in want.items():
             got = torch.frombuffer(bytearray((out / f"{i}.f32").read_bytes()), dtype=torch.float32).view(-1, cfg["vocab"])
             assert _rel(got, ref) < tol, (dtype, i)
+
+
+def test_captured_decoding_runs_the_halves_side_by_side(tmp_path, monkeypatch):
+    """bfloat16 decoding through generate_token: the captured step (mixer and feed-forward as parallel branches of the graph) and the same
+    with one branch after the other choose the same tokens, step for step"""
+    import tgis_b200  # noqa: F401
+    from tgis_b200 import ops_seq, pb
+    cfg = orc.random_config(width=128, heads=8, kv_heads=2, dim=32, vdim=48, rot_dims=16, chunk=60, l_heads=6, l_dim=24, rot_dim=16, l_vdim=40, kv_rank=96,
+                            q_rank=64, experts=6, identity=2, top=3, ff=72, shared=96)
+    model = _model(tmp_path, cfg, orc.random_state_dict(cfg, seed=5), torch.bfloat16, blocks=64, slots=6)
+    forks = []
+    enter = ops_seq.beside.__enter__
+
+    def counting(self):
+        enter(self)
+        forks.append(self.side is not None)
+        return self
+    monkeypatch.setattr(ops_seq.beside, "__enter__", counting)
+    outs = []
+    for on in (True, False):
+        monkeypatch.setattr(ops_seq, "SIDE_STREAM", on)
+        forks.clear()
+        prompts, n_new = [_tokens(60 + i, n, cfg["vocab"]) for i, n in enumerate((9, 40, 77))], 24
+        reqs = [pb.Request(id=i, inputs=" ".join("test" if t == 3 else f"<tok{t}>" for t in p), input_length=len(p), truncate=False, max_output_length=n_new,
+                           parameters=pb.NextTokenChooserParameters(temperature=0.0, top_p=1.0, min_new_tokens=n_new)) for i, p in enumerate(prompts)]
+        got = {i: [] for i in range(3)}
+        with torch.inference_mode():
+            b, errs = model.batch_type.from_pb(pb.Batch(id=0, requests=reqs), model.tokenizer, model.dtype, model.device, None, None, True)
+            assert not errs
+            for step in range(n_new):
+                for t in model.generate_token(b, first=step == 0)[0]:
+                    got[t.request_id].append(t.token_id)
+            model.kv_cache_manager.free_sequences(b.sequence_ids)
+        outs.append(got)
+        assert any(forks) == on
+    assert outs[0] == outs[1] and all(len(v) == 24 for v in outs[0].values())

@@ -235,6 +235,17 @@ __device__ __forceinline__ void ld_vec(const float* p, float (&v)[VEC]) {
     for (int k = 0; k < VEC; ++k) v[k] = p[k];
   }
 }
+template <int VEC>
+__device__ __forceinline__ void ld_vec(const __nv_bfloat16* p, float (&v)[VEC]) {   // VEC 4: 8 bytes
+  if constexpr (VEC == 4) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x)), hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
+  } else {
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) v[k] = ldf(p + k);
+  }
+}
 template <typename T, int VEC>
 __device__ __forceinline__ void st_vec(T* p, const float (&v)[VEC]) {
   if constexpr (VEC == 4 && sizeof(T) == 4) {
@@ -420,7 +431,7 @@ __global__ void __launch_bounds__(kRowThreads) branches_step_kernel(float* __res
 // output the row `pass` that the router read.  One block per token; r waits in shared memory between the passes.
 constexpr int kPicks = 16;
 
-template <typename T, int VEC>
+template <typename T, int VEC, int TOP>   // TOP >= top: the loads of all terms are in flight together
 __global__ void __launch_bounds__(kRowThreads) halves_step_kernel(float* __restrict__ x, const float* __restrict__ init, const float* __restrict__ y1,
                                                                   const float* __restrict__ y2, const float* __restrict__ gate, int64_t ld_gate,
                                                                   const float* __restrict__ rows, int64_t ld_rows, const float* __restrict__ weights,
@@ -432,69 +443,54 @@ __global__ void __launch_bounds__(kRowThreads) halves_step_kernel(float* __restr
   extern __shared__ __align__(16) float row[];
   __shared__ float red[32];
   const int64_t t = blockIdx.x;
+  const float* base = (init ? init : x) + t * W;
   const float s2 = y2 ? (gate ? sigmoid_f(gate[t * ld_gate]) : 1.f) : 0.f;
   // the identity picks share one weight: their row is read once
-  float w_pass = 0.f, w_k[kPicks];
-  const float* src[kPicks];
+  float w_pass = 0.f, w_k[TOP > 0 ? TOP : 1];
+  const float* src[TOP > 0 ? TOP : 1];
 #pragma unroll
-  for (int k = 0; k < kPicks; ++k) {
-    src[k] = nullptr;
-    w_k[k] = 0.f;
-    if (k < top) {
-      const int r = row_of[t * top + k];
-      const float w = weights[t * top + k];
-      if (r >= 0) { src[k] = rows + (int64_t)r * ld_rows; w_k[k] = w; }
-      else w_pass += w;
-    }
+  for (int k = 0; k < TOP; ++k) {
+    const int r = k < top ? row_of[t * top + k] : -1;
+    const float w = k < top ? weights[t * top + k] : 0.f;
+    src[k] = r >= 0 ? rows + (int64_t)r * ld_rows : nullptr;
+    w_k[k] = r >= 0 ? w : 0.f;
+    w_pass += r >= 0 ? 0.f : w;
   }
   float q = 0.f;
   for (int i = threadIdx.x * VEC; i < W; i += kRowThreads * VEC) {
-    float r[VEC], v[VEC];
-    ld_vec<VEC>((init ? init : x) + t * W + i, r);
-    if (y1) {
-      ld_vec<VEC>(y1 + t * W + i, v);
+    float r[VEC], a[VEC] = {}, b[VEC] = {}, h[VEC] = {}, v[TOP > 0 ? TOP : 1][VEC] = {};
+    ld_vec<VEC>(base + i, r);
+    if (y1) ld_vec<VEC>(y1 + t * W + i, a);
+    if (y2) ld_vec<VEC>(y2 + t * W + i, b);
 #pragma unroll
-      for (int k = 0; k < VEC; ++k) r[k] += v[k];
-    }
-    if (y2) {
-      ld_vec<VEC>(y2 + t * W + i, v);
+    for (int e = 0; e < TOP; ++e)
+      if (src[e]) ld_vec<VEC>(src[e] + i, v[e]);
+    if (TOP > 0 && w_pass != 0.f) ld_vec<VEC>(pass + t * W + i, h);
 #pragma unroll
-      for (int k = 0; k < VEC; ++k) r[k] = fmaf(s2, v[k], r[k]);
-    }
-    if (w_pass != 0.f) {
+    for (int k = 0; k < VEC; ++k) {
+      r[k] = fmaf(w_pass, h[k], fmaf(s2, b[k], r[k] + a[k]));
 #pragma unroll
-      for (int k = 0; k < VEC; ++k) r[k] = fmaf(w_pass, ldf(pass + t * W + i + k), r[k]);
-    }
-#pragma unroll
-    for (int e = 0; e < kPicks; ++e) {
-      if (e >= top) break;
-      if (src[e] == nullptr) continue;
-      ld_vec<VEC>(src[e] + i, v);
-#pragma unroll
-      for (int k = 0; k < VEC; ++k) r[k] = fmaf(w_k[e], v[k], r[k]);
+      for (int e = 0; e < TOP; ++e) r[k] = fmaf(w_k[e], v[e][k], r[k]);
+      q += r[k] * r[k];
     }
     st_vec<float, VEC>(x + t * W + i, r);
-    if (norm_a || norm_b) {
-#pragma unroll
-      for (int k = 0; k < VEC; ++k) q += r[k] * r[k];
-      st_vec<float, VEC>(row + i, r);
-    }
+    if (norm_a || norm_b) st_vec<float, VEC>(row + i, r);
   }
   if (!norm_a && !norm_b) return;
   const float rstd = 1.f / sqrtf(block_sum(q, red) / W + eps);
   for (int i = threadIdx.x * VEC; i < W; i += kRowThreads * VEC) {   // every thread reads back what it wrote itself
-    float r[VEC], v[VEC];
+    float r[VEC], wa[VEC] = {}, wb[VEC] = {};
     ld_vec<VEC>(row + i, r);
-    if (norm_a) {
+    if (norm_a) ld_vec<VEC>(norm_a + i, wa);
+    if (norm_b) ld_vec<VEC>(norm_b + i, wb);
 #pragma unroll
-      for (int k = 0; k < VEC; ++k) v[k] = r[k] * rstd * ldf(norm_a + i + k);
-      st_vec<T, VEC>(typed_a + t * W + i, v);
+    for (int k = 0; k < VEC; ++k) {
+      r[k] *= rstd;
+      wa[k] *= r[k];
+      wb[k] *= r[k];
     }
-    if (norm_b) {
-#pragma unroll
-      for (int k = 0; k < VEC; ++k) v[k] = r[k] * rstd * ldf(norm_b + i + k);
-      st_vec<T, VEC>(typed_b + t * W + i, v);
-    }
+    if (norm_a) st_vec<T, VEC>(typed_a + t * W + i, wa);
+    if (norm_b) st_vec<T, VEC>(typed_b + t * W + i, wb);
   }
 }
 
@@ -893,20 +889,31 @@ extern "C" int b200_seq_halves_step(float* x, const float* init, const float* y1
     return B200_ERR_ARG;
   }
   const size_t smem = (size_t)((W + 3) & ~3) * 4;
-#define HST(E, V)                                                                                                                       \
-  do {                                                                                                                                  \
-    static bool cfg = false;                                                                                                            \
-    if (!cfg) { cudaFuncSetAttribute(halves_step_kernel<E, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024); cfg = true; }  \
-    B200_LAUNCH((halves_step_kernel<E, V>), dim3((unsigned)T), dim3(kRowThreads), smem, (cudaStream_t)stream, x, init, y1, y2, gate, ld_gate, rows, \
+#define HST_TOP(E, V, N)                                                                                                                 \
+  do {                                                                                                                                   \
+    static bool cfg = false;                                                                                                             \
+    if (!cfg) { cudaFuncSetAttribute(halves_step_kernel<E, V, N>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024); cfg = true; } \
+    B200_LAUNCH((halves_step_kernel<E, V, N>), dim3((unsigned)T), dim3(kRowThreads), smem, (cudaStream_t)stream, x, init, y1, y2, gate, ld_gate, rows, \
                 ld_rows, weights, row_of, top, (const E*)pass, (const E*)norm_a, (const E*)norm_b, (E*)typed_a, (E*)typed_b, (int)W, eps); \
+  } while (0)
+#define HST(E)                          \
+  do {                                  \
+    if (!vec) HST_TOP(E, 1, kPicks);    \
+    else if (top == 0) HST_TOP(E, 4, 0); \
+    else if (top <= 2) HST_TOP(E, 4, 2); \
+    else if (top <= 4) HST_TOP(E, 4, 4); \
+    else if (top <= 8) HST_TOP(E, 4, 8); \
+    else HST_TOP(E, 4, kPicks);         \
   } while (0)
   const bool vec = W % 4 == 0 && ld_rows % 4 == 0 &&
                    ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(init) | reinterpret_cast<uintptr_t>(y1) | reinterpret_cast<uintptr_t>(y2) |
-                     reinterpret_cast<uintptr_t>(rows) | reinterpret_cast<uintptr_t>(typed_a) | reinterpret_cast<uintptr_t>(typed_b)) & 15) == 0;
-  if (dt == B200_DT_F32) { if (vec) HST(float, 4); else HST(float, 1); }
-  else if (dt == B200_DT_BF16) { if (vec) HST(__nv_bfloat16, 4); else HST(__nv_bfloat16, 1); }
+                     reinterpret_cast<uintptr_t>(rows) | reinterpret_cast<uintptr_t>(typed_a) | reinterpret_cast<uintptr_t>(typed_b) |
+                     reinterpret_cast<uintptr_t>(pass) | reinterpret_cast<uintptr_t>(norm_a) | reinterpret_cast<uintptr_t>(norm_b)) & 15) == 0;
+  if (dt == B200_DT_F32) HST(float);
+  else if (dt == B200_DT_BF16) HST(__nv_bfloat16);
   else { b200_set_last_error("unknown element type"); return B200_ERR_ARG; }
 #undef HST
+#undef HST_TOP
   b200_count_launches(1);
   return B200_OK;
 }

@@ -150,14 +150,17 @@ class TibopelLayer(nn.Module):
             self.norm2 = weights.get_tensor(f"{pre}.norm2").contiguous()
 
     def halves(self, h1: torch.Tensor, h2: Optional[torch.Tensor], step: ops.RaggedStep, manager: HybridCacheManager, max_s: int) -> Dict[str, Any]:
-        """what the layer adds to the stream, as arguments of `ops.halves_step`"""
+        """what the layer adds to the stream, as arguments of `ops.halves_step`; in a captured decoding step the two halves run side by side"""
+        out: Dict[str, Any] = {}
+        with ops.beside(h1.device) as side:
+            if self.mlp is not None:
+                out.update(self.mlp(h2))
         if isinstance(self.mixer, LatentAttention):
             y = self.mixer(h1, step, manager.layer_pages(self.index), max_s)
         else:
             y = self.mixer(h1, step, manager.layer_pages(self.index), None, max_s)
-        out = {"y1": y}
-        if self.mlp is not None:
-            out.update(self.mlp(h2))
+        side.join()
+        out["y1"] = y
         return out
 
 

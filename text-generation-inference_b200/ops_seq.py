@@ -58,16 +58,62 @@ class RaggedStep:
 _TC_GEMM = os.getenv("B200_SEQ_TC_GEMM", "1") != "0"
 _ATTN_SPLIT = os.getenv("B200_SEQ_ATTN_SPLIT", "1") != "0"
 _gemm_ws = {}
+_side_streams = {}
+_on_side = False
+SIDE_STREAM = os.getenv("B200_SEQ_SIDE_STREAM", "1") != "0"
 
 
-def _gemm_workspace(device, N: int, K: int) -> torch.Tensor:
-    """per-device split-K workspace of the tensor-core product (tile counters zeroed once; the kernel re-arms them)"""
+def _gemm_workspace(device, N: int, K: int, side: Optional[bool] = None) -> torch.Tensor:
+    """split-K workspace of the tensor-core product, one per device and stream that products run on side by side (tile counters zeroed
+    once; the kernel re-arms them)"""
     need = _lib.load_seq().b200_gemm_workspace_bytes_max(N, K)
-    ws = _gemm_ws.get(device)
+    key = (device, _on_side if side is None else side)
+    ws = _gemm_ws.get(key)
     if ws is None or ws.numel() < need:
         ws = torch.zeros(max(need, 1 << 20), dtype=torch.uint8, device=device)
-        _gemm_ws[device] = ws
+        _gemm_ws[key] = ws
     return ws
+
+
+class beside:
+    """`with beside(device) as s:` queues what is inside on a second stream, behind everything queued so far; `s.join()` makes the current
+    stream wait for it.  Only while a CUDA graph is captured: there the two branches become parallel parts of the graph, so that the
+    short launches of two independent halves of a decoding layer overlap.  Elsewhere (eager steps are bound by the host, prompts fill
+    the device) the block simply runs in place.  What the block reads must stay referenced until the join; the workspaces of its products
+    must have been reserved (`reserve_side_workspace`), since a graph must not hold the call that zeroes one."""
+
+    def __init__(self, device):
+        self.device, self.side = torch.device(device), None
+
+    def __enter__(self):
+        global _on_side
+        if SIDE_STREAM and not _on_side and torch.cuda.is_current_stream_capturing():
+            self.side = _side_streams.setdefault(self.device, torch.cuda.Stream(self.device))
+            self.side.wait_stream(torch.cuda.current_stream(self.device))
+            self.ctx = torch.cuda.stream(self.side)
+            self.ctx.__enter__()
+            _on_side = True
+        return self
+
+    def __exit__(self, *exc):
+        global _on_side
+        if self.side is not None:
+            _on_side = False
+            self.ctx.__exit__(*exc)
+        return False
+
+    def join(self) -> None:
+        if self.side is not None:
+            torch.cuda.current_stream(self.device).wait_stream(self.side)
+            self.side = None
+
+
+def reserve_side_workspace(device, shapes) -> None:
+    """workspace of the products (N, K) that will run inside `beside`"""
+    if torch.device(device).type == "cuda":
+        _side_streams.setdefault(torch.device(device), torch.cuda.Stream(device))
+        for n, k in shapes:
+            _gemm_workspace(torch.device(device), n, k, side=True)
 
 
 ACT_SILU, ACT_GELU_TANH, ACT_TANH, ACT_RELU2, ACT_NONE = 0, 1, 2, 3, 4

@@ -391,6 +391,8 @@ class RoutedSharedFeedForward(nn.Module):
         self.routed = RoutedExperts(prefix, weights, experts=experts, top=top, limit=None, softmax_scores=True, correction=True, identity=identity,
                                     plain="relu2", more_rows=gate_row)
         self.shared = PlainMLP(f"{prefix}.shared", weights, activation="relu2") if shared else None
+        dense = [self.routed.w_router] + ([self.shared.w_up, self.shared.w_down] if shared else [])
+        ops.reserve_side_workspace(self.routed.w_router.device, [w.shape for w in dense])     # may run beside the mixer
 
     def forward(self, h: torch.Tensor) -> dict:
         routing, more = self.routed.route(h)
