@@ -280,14 +280,32 @@ __global__ void __launch_bounds__(kTileThreads) latent_attn_tile_kernel(
     float s[2][4] = {};
     if (s_warp) {
       const uint32_t b_lane = k_stage + (uint32_t)(((kg * 16 + (lm >> 1) * 8 + lr) * DP + (lm & 1) * 8) * 2);
-#pragma unroll 4
-      for (int kk = 0; kk < D; kk += 16) {
-        uint32_t a[4], bb[4];
-        ldmatrix_x4(a[0], a[1], a[2], a[3], a_lane + kk * 2);
-        ldmatrix_x4(bb[0], bb[1], bb[2], bb[3], b_lane + kk * 2);
-        mma_m16n8k16_bf16f32(s[0], a, bb[0], bb[1]);
-        mma_m16n8k16_bf16f32(s[1], a, bb[2], bb[3]);
+      // two sets of accumulators and four k-steps of fragments at a time: the products of a warp must not wait for one another
+      float s2[2][4] = {};
+      uint32_t a[4][4], bb[4][4];
+      int kk = 0;
+      for (; kk + 64 <= D; kk += 64) {
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          ldmatrix_x4(a[u][0], a[u][1], a[u][2], a[u][3], a_lane + (kk + u * 16) * 2);
+          ldmatrix_x4(bb[u][0], bb[u][1], bb[u][2], bb[u][3], b_lane + (kk + u * 16) * 2);
+        }
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+          mma_m16n8k16_bf16f32(u & 1 ? s2[0] : s[0], a[u], bb[u][0], bb[u][1]);
+          mma_m16n8k16_bf16f32(u & 1 ? s2[1] : s[1], a[u], bb[u][2], bb[u][3]);
+        }
       }
+      for (; kk < D; kk += 16) {
+        ldmatrix_x4(a[0][0], a[0][1], a[0][2], a[0][3], a_lane + kk * 2);
+        ldmatrix_x4(bb[0][0], bb[0][1], bb[0][2], bb[0][3], b_lane + kk * 2);
+        mma_m16n8k16_bf16f32(s[0], a[0], bb[0][0], bb[0][1]);
+        mma_m16n8k16_bf16f32(s[1], a[0], bb[0][2], bb[0][3]);
+      }
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[nt][e] += s2[nt][e];
       float mx[2] = {-INFINITY, -INFINITY};
       const bool interior = j0 + KT - 1 <= min(j_end, p_first) && j0 >= lo_last;   // every key is visible to every row
 #pragma unroll
@@ -355,17 +373,22 @@ __global__ void __launch_bounds__(kTileThreads) latent_attn_tile_kernel(
         uint32_t a[PRT][4];
 #pragma unroll
         for (int t = 0; t < PRT; ++t) ldmatrix_x4(a[t][0], a[t][1], a[t][2], a[t][3], p_lane + (uint32_t)((t * 16 * PP + ks * 16) * 2));
+        constexpr int NF = NP < 4 ? NP : 4;   // pieces whose fragments are fetched together
 #pragma unroll
-        for (int i = 0; i < NP; ++i) {
-          if (pc + i * PC < pieces) {
-            uint32_t bb[4];
-            ldmatrix_x4_trans(bb[0], bb[1], bb[2], bb[3], v_lane + (uint32_t)((ks * 16 * DP + i * PC * 16) * 2));
+        for (int i0 = 0; i0 < NP; i0 += NF) {
+          uint32_t bb[NF][4];
 #pragma unroll
-            for (int t = 0; t < PRT; ++t) {
-              mma_m16n8k16_bf16f32(o[t][2 * i], a[t], bb[0], bb[1]);
-              mma_m16n8k16_bf16f32(o[t][2 * i + 1], a[t], bb[2], bb[3]);
-            }
-          }
+          for (int i = 0; i < NF; ++i)
+            if (pc + (i0 + i) * PC < pieces)
+              ldmatrix_x4_trans(bb[i][0], bb[i][1], bb[i][2], bb[i][3], v_lane + (uint32_t)((ks * 16 * DP + (i0 + i) * PC * 16) * 2));
+#pragma unroll
+          for (int i = 0; i < NF; ++i)
+            if (pc + (i0 + i) * PC < pieces)
+#pragma unroll
+              for (int t = 0; t < PRT; ++t) {
+                mma_m16n8k16_bf16f32(o[t][2 * (i0 + i)], a[t], bb[i][0], bb[i][1]);
+                mma_m16n8k16_bf16f32(o[t][2 * (i0 + i) + 1], a[t], bb[i][2], bb[i][3]);
+              }
         }
       }
     }
