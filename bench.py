@@ -1471,8 +1471,10 @@ def run_tibopel_compare(args):
         # the picks that are experts (identity outputs cost nothing): counted in the prefill that was timed
         rows = r["pre_rows"]
         lin_flops, moe_flops = 2 * T * dense_w + 2 * PB * head_w, 2 * rows * expert_w
-        # a layer's boundary: stream in and out, the mixer's and the shared expert's results, the picked rows, the passed row, two typed rows out
-        stream_b = sum(width * (8 + 4 + 4 + 4 * top + 2 + 4) for _ in L)
+        # a layer's boundary: stream in and out, the mixer's and the shared expert's results, two typed rows out (not after the last layer); the
+        # picks' rows, 4 bytes per column for an expert's, 2 for the passed one
+        stream_b = width * (12 + 4 + (len(L) - 1) * (8 + 8 + 4) + 8 + 8)
+        pick_b = width * (4 * rows + 2 * (T * len(L) * top - rows))
         a_us, m_us, g_us, h_us = us(dk, "talk_attn"), us(dk, "moe_linear"), dk.get("gemm_f16_kernel", 0.0), us(dk, "halves_step")
         kernels = {
             "talk_attn prefill": {"ms": pre["talk_attn"], "tflops": attn_flops / pre["talk_attn"] / 1e9,
@@ -1483,8 +1485,9 @@ def run_tibopel_compare(args):
             "linear decode (tcgen05 projections)": {"us": g_us, "of_measured_hbm": (dense_w + head_w) * 2 / (max(g_us, 1e-9) * 1e-6) / hbm},
             "moe_linear decode (grouped, picked experts' weights once)": {"us": m_us, "experts_picked_all_layers": r["picked"], "of_measured_hbm":
                                                                           r["picked"] * expert_w * 2 / (max(m_us, 1e-9) * 1e-6) / hbm},
-            "halves_step prefill": {"ms": pre["halves_step"], "of_measured_hbm": T * stream_b / (pre["halves_step"] * 1e-3) / hbm},
-            "halves_step decode": {"us": h_us, "launches": len(L) + 1, "of_measured_hbm": DB * stream_b / (max(h_us, 1e-9) * 1e-6) / hbm},
+            "halves_step prefill": {"ms": pre["halves_step"], "of_measured_hbm": (T * stream_b + pick_b) / (pre["halves_step"] * 1e-3) / hbm},
+            "halves_step decode": {"us": h_us, "launches": len(L) + 1, "of_measured_hbm":
+                                   DB * (stream_b + pick_b / T) / (max(h_us, 1e-9) * 1e-6) / hbm},
         }
         kernels["experts_linear prefill (grouped)"] = {"ms": pre["experts_linear"], "rows": rows,
                                                        "of_measured_tensor": moe_flops / (pre["experts_linear"] * 1e-3) / tens}

@@ -57,6 +57,32 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return warp_sum(t);
 }
 
+// Ragged steps cut into tiles: sequence b has ceil((cu_q[b + 1] - cu_q[b]) * per_token / rows) tiles of `rows` rows.  Which sequence number
+// `tile` falls to (`b`; B: none, there are fewer tiles), and its number among that sequence's tiles (`tile`).  All lanes of a warp call
+// it with the same arguments: 32 sequences at a time, a lane each.
+__device__ __forceinline__ void find_ragged_tile(const int32_t* cu_q, int B, int per_token, int rows, int& b, int& tile) {
+  const int lane = lane_id();
+  for (int b0 = 0; b0 < B; b0 += 32) {
+    const int n = b0 + lane < B ? (cu_q[b0 + lane + 1] - cu_q[b0 + lane]) * per_token : 0;
+    const int nt = (n + rows - 1) / rows;
+    int upto = nt;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int v = __shfl_up_sync(0xffffffffu, upto, o);
+      if (lane >= o) upto += v;
+    }
+    const unsigned hit = __ballot_sync(0xffffffffu, tile < upto);
+    if (hit) {
+      const int at = __ffs(hit) - 1;
+      b = b0 + at;
+      tile -= __shfl_sync(0xffffffffu, upto - nt, at);
+      return;
+    }
+    tile -= __shfl_sync(0xffffffffu, upto, 31);
+  }
+  b = B;
+}
+
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }

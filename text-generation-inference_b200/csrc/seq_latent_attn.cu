@@ -175,15 +175,11 @@ struct LatentTile {
 
 // which (sequence, tile of `rows` of its (token, head) rows) block `tile` has, a sequence's last tile first; b == B: none
 __device__ __forceinline__ void latent_find_tile(const int32_t* cu_q, int B, int H, int rows, int tile, int& b, int& first, int& n_rows) {
-  for (b = 0; b < B; ++b) {
-    const int n = (cu_q[b + 1] - cu_q[b]) * H, nt = (n + rows - 1) / rows;
-    if (tile < nt) {
-      first = (nt - 1 - tile) * rows;   // the last rows see the most keys: they start first
-      n_rows = min(rows, n - first);
-      return;
-    }
-    tile -= nt;
-  }
+  find_ragged_tile(cu_q, B, H, rows, b, tile);
+  if (b >= B) return;
+  const int n = (cu_q[b + 1] - cu_q[b]) * H, nt = (n + rows - 1) / rows;
+  first = (nt - 1 - tile) * rows;   // the last rows see the most keys: they start first
+  n_rows = min(rows, n - first);
 }
 
 template <typename T>
@@ -439,41 +435,45 @@ __global__ void __launch_bounds__(kTileThreads) latent_attn_tile_kernel(
     }
 }
 
-// out[row] = sum_z 2^(m_z - M) O_z / sum_z 2^(m_z - M) l_z over the key runs of latent_attn_tile_kernel; one warp per row, blocks (tile, 8 rows)
+// out[row] = sum_z 2^(m_z - M) O_z / sum_z 2^(m_z - M) l_z over the key runs of latent_attn_tile_kernel; a block per row, two columns per
+// thread, the runs' loads in flight together (NS >= nsplit: runs past the last read the last again, with no weight)
 constexpr int kLatentRuns = 16;
 
+template <int NS>
 __global__ void __launch_bounds__(256) latent_attn_merge_kernel(const float* __restrict__ partial, __nv_bfloat16* __restrict__ out,
                                                                 const int32_t* __restrict__ cu_q, int B, int H, int R, int rows, int nsplit) {
   pdl_launch_dependents();
   pdl_wait();
   int b, first = 0, n_rows = 0;
   latent_find_tile(cu_q, B, H, rows, blockIdx.x, b, first, n_rows);
-  const int row = blockIdx.y * 8 + warp_id(), lane = lane_id();
+  const int row = blockIdx.y;
   if (b >= B || row >= n_rows) return;
   const float* base = partial + ((int64_t)blockIdx.x * nsplit * rows + row) * (R + 2);
   const int64_t zs = (int64_t)rows * (R + 2);
-  float M = -INFINITY, wz[kLatentRuns], den = 0.f;
+  float wz[NS], lz[NS], M = -INFINITY, den = 0.f;
 #pragma unroll
-  for (int z = 0; z < kLatentRuns; ++z) {
-    wz[z] = z < nsplit ? base[z * zs + R] : -INFINITY;
+  for (int z = 0; z < NS; ++z) {
+    const float2 ml = *reinterpret_cast<const float2*>(base + min(z, nsplit - 1) * zs + R);
+    wz[z] = z < nsplit ? ml.x : -INFINITY;
+    lz[z] = ml.y;
     M = fmaxf(M, wz[z]);
   }
 #pragma unroll
-  for (int z = 0; z < kLatentRuns; ++z) {
+  for (int z = 0; z < NS; ++z) {
     wz[z] = wz[z] > -INFINITY ? exp2f(wz[z] - M) : 0.f;  // an empty run carries no weight
-    if (z < nsplit) den += wz[z] * base[z * zs + R + 1];
+    den = fmaf(wz[z], lz[z], den);
   }
   const float inv = 1.f / den;
   const int64_t dst = ((int64_t)cu_q[b] * H + first + row) * R;
-  for (int c = lane * 2; c < R; c += 64) {
-    float2 acc = make_float2(0.f, 0.f);
+  for (int c = threadIdx.x * 2; c < R; c += blockDim.x * 2) {
+    float2 v[NS], acc = make_float2(0.f, 0.f);
 #pragma unroll
-    for (int z = 0; z < kLatentRuns; ++z)
-      if (z < nsplit) {
-        const float2 v = *reinterpret_cast<const float2*>(base + z * zs + c);
-        acc.x = fmaf(wz[z], v.x, acc.x);
-        acc.y = fmaf(wz[z], v.y, acc.y);
-      }
+    for (int z = 0; z < NS; ++z) v[z] = *reinterpret_cast<const float2*>(base + min(z, nsplit - 1) * zs + c);
+#pragma unroll
+    for (int z = 0; z < NS; ++z) {
+      acc.x = fmaf(wz[z], v[z].x, acc.x);
+      acc.y = fmaf(wz[z], v[z].y, acc.y);
+    }
     latent_store<__nv_bfloat16>(out, dst + c, acc.x * inv, acc.y * inv);
   }
 }
@@ -585,9 +585,14 @@ extern "C" int b200_seq_latent_attn(const void* q_abs, const void* cache, int dt
       else LAT(1, 4);
     }
 #undef LAT
-    if (nsplit > 1)
-      B200_LAUNCH(latent_attn_merge_kernel, dim3((unsigned)tiles, (unsigned)(rows / 8)), dim3(256), 0, st, (const float*)partial, (__nv_bfloat16*)out, cu_q,
-                  B, H, R, (int)rows, nsplit);
+#define MERGE(NS)                                                                                                                        \
+  B200_LAUNCH(latent_attn_merge_kernel<NS>, dim3((unsigned)tiles, (unsigned)rows), dim3(R > 256 ? 256 : R > 128 ? 128 : 64), 0, st,       \
+              (const float*)partial, (__nv_bfloat16*)out, cu_q, B, H, R, (int)rows, nsplit)
+    if (nsplit > 8) MERGE(16);
+    else if (nsplit > 4) MERGE(8);
+    else if (nsplit > 2) MERGE(4);
+    else if (nsplit > 1) MERGE(2);
+#undef MERGE
     b200_count_launches(nsplit > 1 ? 2 : 1);
     return B200_OK;
   }

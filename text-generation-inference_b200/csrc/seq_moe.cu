@@ -52,13 +52,13 @@ __host__ __device__ inline MoePlan moe_plan_view(int32_t* base, int64_t T, int E
 }
 
 // One warp: the `top` picks of one token from its E router outputs (fp32) and their weights; `took(k, e)` runs in lane 0 for every pick
-template <int MODE, typename Took>
+template <int MODE, int PER, typename Took>   // PER: router outputs per lane, at most
 __device__ __forceinline__ void moe_pick(const float* __restrict__ row, int E, int top, const void* __restrict__ correction, int corr_dt,
                                          float weight_scale, float* __restrict__ w_out, Took took) {
   const int lane = lane_id();
-  float z[kMaxExpertsPerLane], sc[kMaxExpertsPerLane];
+  float z[PER], sc[PER];
 #pragma unroll
-  for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+  for (int i = 0; i < PER; ++i) {
     const int e = lane + 32 * i;
     z[i] = e < E ? row[e] : -INFINITY;
     sc[i] = 0.f;
@@ -67,20 +67,20 @@ __device__ __forceinline__ void moe_pick(const float* __restrict__ row, int E, i
   if (MODE == 2) {  // soft-max over all router outputs
     float m = z[0], sum = 0.f;
 #pragma unroll
-    for (int i = 1; i < kMaxExpertsPerLane; ++i) m = fmaxf(m, z[i]);
+    for (int i = 1; i < PER; ++i) m = fmaxf(m, z[i]);
     m = warp_max(m);
 #pragma unroll
-    for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+    for (int i = 0; i < PER; ++i) {
       sc[i] = lane + 32 * i < E ? expf(z[i] - m) : 0.f;
       sum += sc[i];
     }
     const float inv = 1.f / warp_sum(sum);
 #pragma unroll
-    for (int i = 0; i < kMaxExpertsPerLane; ++i) sc[i] *= inv;
+    for (int i = 0; i < PER; ++i) sc[i] *= inv;
   }
   if (MODE != 0) {
 #pragma unroll
-    for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+    for (int i = 0; i < PER; ++i) {
       const int e = lane + 32 * i;
       if (e < E) z[i] = sc[i] + (correction ? ld_any(correction, e, corr_dt) : 0.f);
     }
@@ -93,7 +93,7 @@ __device__ __forceinline__ void moe_pick(const float* __restrict__ row, int E, i
     float best = -INFINITY;
     int be = 0x7fffffff;
 #pragma unroll
-    for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+    for (int i = 0; i < PER; ++i) {
       const int e = lane + 32 * i;
       if (e < E && (z[i] > best || (z[i] == best && e < be))) { best = z[i]; be = e; }
     }
@@ -107,14 +107,14 @@ __device__ __forceinline__ void moe_pick(const float* __restrict__ row, int E, i
     if (MODE != 0) {  // the weight uses the plain score of the pick, which its owning lane holds
       float mine = 0.f;
 #pragma unroll
-      for (int i = 0; i < kMaxExpertsPerLane; ++i)
+      for (int i = 0; i < PER; ++i)
         if (lane + 32 * i == be) mine = sc[i];
       best = __shfl_sync(0xffffffffu, mine, be & 31);
     }
     val[k] = best;
     idx[k] = be;
 #pragma unroll
-    for (int i = 0; i < kMaxExpertsPerLane; ++i)
+    for (int i = 0; i < PER; ++i)
       if (lane + 32 * i == be) z[i] = -INFINITY;
   }
   if (lane == 0) {
@@ -179,7 +179,7 @@ __device__ __forceinline__ void moe_offsets(const int* counts, int* offs, int E,
 
 // picks of the whole step, 8 tokens per block; the places in the experts' lists come from counters in the plan.  Router outputs from E
 // on (up to E_all) are identity outputs: they are picked like experts but take no row (place -1).
-template <int MODE>
+template <int MODE, int PER>
 __global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict__ logits, int64_t ld, int64_t T, int E, int E_all, int top,
                                                         int32_t* __restrict__ ids, float* __restrict__ weights, MoePlan p,
                                                         const void* __restrict__ correction, int corr_dt, float weight_scale) {
@@ -187,7 +187,7 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict_
   pdl_wait();
   const int64_t t = (int64_t)blockIdx.x * 8 + warp_id();
   if (t >= T) return;
-  moe_pick<MODE>(logits + t * ld, E_all, top, correction, corr_dt, weight_scale, weights + t * top, [&](int k, int e) {
+  moe_pick<MODE, PER>(logits + t * ld, E_all, top, correction, corr_dt, weight_scale, weights + t * top, [&](int k, int e) {
     ids[t * top + k] = e;
     p.place[t * top + k] = e < E ? atomicAdd(p.counts + e, 1) : -1;
   });
@@ -211,7 +211,7 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const int32_t* __restric
 // picks and plan of a step of few tokens (decoding) in one launch: one block, counters in shared memory
 constexpr int kRouteOnePass = 64;
 
-template <int MODE>
+template <int MODE, int PER>
 __global__ void __launch_bounds__(1024) moe_route_plan_kernel(const float* __restrict__ logits, int64_t ld, int T, int E, int E_all, int top,
                                                               int32_t* __restrict__ ids, float* __restrict__ weights, MoePlan p,
                                                               const void* __restrict__ correction, int corr_dt, float weight_scale) {
@@ -222,7 +222,7 @@ __global__ void __launch_bounds__(1024) moe_route_plan_kernel(const float* __res
   __syncthreads();
   pdl_wait();
   for (int t = warp_id(); t < T; t += blockDim.x / 32)
-    moe_pick<MODE>(logits + t * ld, E_all, top, correction, corr_dt, weight_scale, weights + t * top, [&](int k, int e) {
+    moe_pick<MODE, PER>(logits + t * ld, E_all, top, correction, corr_dt, weight_scale, weights + t * top, [&](int k, int e) {
       s_id[t * top + k] = e;
       s_place[t * top + k] = e < E ? atomicAdd(counts + e, 1) : -1;
     });
@@ -434,24 +434,31 @@ extern "C" int b200_seq_moe_route_scored(const float* logits, int64_t ld, int64_
   }
   cudaStream_t st = (cudaStream_t)stream;
   MoePlan p = moe_plan_view(plan, T, E, top);
-#define ROUTE(M)                                                                                                                          \
-  do {                                                                                                                                    \
-    if (T <= kRouteOnePass) {                                                                                                             \
-      B200_LAUNCH(moe_route_plan_kernel<M>, dim3(1), dim3(T <= 8 ? 256 : 1024), 0, st, logits, ld, (int)T, E, E_all, top, ids, weights, p, \
-                  correction, corr_dt, weight_scale);                                                                                     \
-      b200_count_launches(1);                                                                                                             \
-      return B200_OK;                                                                                                                     \
-    }                                                                                                                                     \
-    if (cudaMemsetAsync(p.counts, 0, sizeof(int32_t) * E, st) != cudaSuccess) { b200_set_last_error("seq_moe_route: memset failed"); return B200_ERR_CUDA; } \
-    B200_LAUNCH(moe_route_kernel<M>, dim3((unsigned)((T + 7) / 8)), dim3(256), 0, st, logits, ld, T, E, E_all, top, ids, weights, p, correction, \
-                corr_dt, weight_scale);                                                                                                   \
+  const bool one_pass = T <= kRouteOnePass;
+  if (!one_pass && cudaMemsetAsync(p.counts, 0, sizeof(int32_t) * E, st) != cudaSuccess) { b200_set_last_error("seq_moe_route: memset failed"); return B200_ERR_CUDA; }
+#define ROUTE(M, PER)                                                                                                                          \
+  do {                                                                                                                                         \
+    if (one_pass)                                                                                                                              \
+      B200_LAUNCH((moe_route_plan_kernel<M, PER>), dim3(1), dim3(T <= 8 ? 256 : 1024), 0, st, logits, ld, (int)T, E, E_all, top, ids, weights, p, \
+                  correction, corr_dt, weight_scale);                                                                                          \
+    else                                                                                                                                       \
+      B200_LAUNCH((moe_route_kernel<M, PER>), dim3((unsigned)((T + 7) / 8)), dim3(256), 0, st, logits, ld, T, E, E_all, top, ids, weights, p,   \
+                  correction, corr_dt, weight_scale);                                                                                          \
   } while (0)
-  if (mode == 2) ROUTE(2);
-  else if (mode == 1) ROUTE(1);
-  else ROUTE(0);
+  if (E_all <= 32) {
+    if (mode == 2) ROUTE(2, 1);
+    else if (mode == 1) ROUTE(1, 1);
+    else ROUTE(0, 1);
+  } else {
+    if (mode == 2) ROUTE(2, kMaxExpertsPerLane);
+    else if (mode == 1) ROUTE(1, kMaxExpertsPerLane);
+    else ROUTE(0, kMaxExpertsPerLane);
+  }
 #undef ROUTE
+  b200_count_launches(1);
+  if (one_pass) return B200_OK;
   B200_LAUNCH(moe_plan_kernel, dim3(1), dim3(1024), 0, st, (const int32_t*)ids, T * top, top, E, p);
-  b200_count_launches(2);
+  b200_count_launches(1);
   return B200_OK;
 }
 

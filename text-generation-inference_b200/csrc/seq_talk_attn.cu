@@ -290,16 +290,10 @@ __device__ __forceinline__ void ffma2(float2& acc, float t, float vx, float vy) 
 
 // which (sequence, tile of QT of its rows) block `tile` has; b == B: none
 __device__ __forceinline__ void talk_find_tile(const int32_t* cu_q, int B, int QT, int tile, int& b, int& row0, int& ntok) {
-  for (b = 0; b < B; ++b) {
-    const int n = cu_q[b + 1] - cu_q[b];
-    const int nt = (n + QT - 1) / QT;
-    if (tile < nt) {
-      row0 = cu_q[b] + tile * QT;
-      ntok = min(QT, cu_q[b + 1] - row0);
-      return;
-    }
-    tile -= nt;
-  }
+  find_ragged_tile(cu_q, B, 1, QT, b, tile);
+  if (b >= B) return;
+  row0 = cu_q[b] + tile * QT;
+  ntok = min(QT, cu_q[b + 1] - row0);
 }
 
 template <int NDV, int KT>  // NDV = vdim / 8 output n-tiles per warp, KT keys per tile
