@@ -905,8 +905,8 @@ def run_hybrid_compare(args):
         kernels = {
             "latent_attn prefill": {"ms": pre_ops["latent_attn"], "tflops": attn_flops / pre_ops["latent_attn"] / 1e9,
                                     "of_measured_tensor": attn_flops / (pre_ops["latent_attn"] * 1e-3) / tens},
-            "latent_attn decode": {"us": dec_k.get("latent_attn_mma_kernel", 0.0) + dec_k.get("latent_attn_merge_kernel", 0.0), "of_measured_hbm":
-                                   DB * ctx * D * 2 / ((dec_k.get("latent_attn_mma_kernel", 0.0) + dec_k.get("latent_attn_merge_kernel", 0.0)) * 1e-6) / hbm},
+            "latent_attn decode": {"us": dec_k.get("latent_attn_tile_kernel", 0.0) + dec_k.get("latent_attn_merge_kernel", 0.0), "of_measured_hbm":
+                                   DB * ctx * D * 2 / ((dec_k.get("latent_attn_tile_kernel", 0.0) + dec_k.get("latent_attn_merge_kernel", 0.0)) * 1e-6) / hbm},
             "ssm_scan decode": {"us": dec_k["ssm_scan_kernel"], "of_measured_hbm":
                                 DB * ss["heads"] * ss["state"] * ss["vdim"] * 8 / (dec_k["ssm_scan_kernel"] * 1e-6) / hbm},
             "mlstm_scan decode": {"us": dec_k["mlstm_scan_kernel"], "of_measured_hbm":
